@@ -12,7 +12,8 @@ class KVRequest:
     """Keys and values of every position (window and chunk None), of the last ``window`` positions, or of the chunk of
     ``chunk`` positions that the newest position lies in (chunks counted from position 0).  ``keep_first``: with a window,
     the sequence's first ``keep_first`` positions are kept for good as well.  ``values_are_keys``: the mixer's values are
-    its keys as cached, so the pages hold keys alone and the view's value pages are the key pages."""
+    its keys as cached (with ``v_head_dim``: their first ``v_head_dim`` numbers), so the pages hold keys alone and the view's
+    value pages are the key pages, or a view of them."""
     n_kv_heads: int
     head_dim: int
     window: Optional[int] = None
@@ -22,8 +23,8 @@ class KVRequest:
     values_are_keys: bool = False
 
     def __post_init__(self):
-        if self.values_are_keys and self.v_head_dim is not None and self.v_head_dim != self.head_dim:
-            raise ValueError("keys that serve as values have one size")
+        if self.values_are_keys and self.v_head_dim is not None and self.v_head_dim > self.head_dim:
+            raise ValueError("values that lie inside the keys cannot be wider than they")
         if self.window and self.chunk:
             raise ValueError("a cache request keeps a window or a chunk, not both")
         if self.keep_first < 0 or (self.keep_first and not self.window):
@@ -46,9 +47,11 @@ class KVRequest:
 class StateRequest:
     """Per-sequence state of fixed size: {name: (shape, dtype)}; zero when a slot is handed out.
 
-    dtype None means the model's compute dtype.
+    dtype None means the model's compute dtype.  ``repeatable``: a step of one token per sequence that is run again (with other
+    tokens) leaves the state as if it had run once, so that steps may be launched ahead of the host and dropped.
     """
     tensors: Tuple[Tuple[str, Tuple[int, ...], Optional[torch.dtype]], ...]
+    repeatable: bool = False
 
     @staticmethod
     def of(**named) -> "StateRequest":

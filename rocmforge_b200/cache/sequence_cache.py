@@ -45,8 +45,8 @@ class KVGroup:
         self.pool = FreeList(n_pages, "cache page")
         # [owner, k|v, page, kv_head, position in page, head_dim]; values of another head size than keys have a tensor
         # of their own (storage then holds the keys alone)
-        self.separate_values = request.v_head_dim is not None and request.v_head_dim != request.head_dim
-        self.keys_only = bool(request.values_are_keys)             # the values are the keys: one plane, read twice
+        self.keys_only = bool(request.values_are_keys)             # the values are (part of) the keys: one plane, read twice
+        self.separate_values = not self.keys_only and request.v_head_dim is not None and request.v_head_dim != request.head_dim
         self.storage = torch.zeros((len(self.owners), 1 if self.separate_values or self.keys_only else 2, n_pages, request.n_kv_heads, PAGE,
                                     request.head_dim), dtype=dtype, device=device)
         self.value_storage = (torch.zeros((len(self.owners), 1, n_pages, request.n_kv_heads, PAGE, request.v_head_dim),
@@ -153,7 +153,11 @@ class KVGroup:
     def v_pages(self, owner: int) -> torch.Tensor:
         if self.separate_values:
             return self.value_storage[self.index_of[owner], 0]
-        return self.storage[self.index_of[owner], 0 if self.keys_only else 1]
+        if self.keys_only:
+            pages = self.storage[self.index_of[owner], 0]
+            vd = self.request.v_head_dim
+            return pages if vd is None or vd == self.request.head_dim else pages[..., :vd]
+        return self.storage[self.index_of[owner], 1]
 
 
 @dataclass
@@ -204,6 +208,9 @@ class SequenceCache:
         by_key: Dict[tuple, List[int]] = {}
         self._kv_request: Dict[tuple, KVRequest] = {}
         self.states: Dict[int, StateView] = {}
+        # whether a step of one token per sequence may run twice (pages: written again with the same positions; state: only if
+        # its owner says so)
+        self.steps_repeatable = True
         # a mixer made of several (side by side) asks with a dict {name: request}: every entry is kept under the
         # owner (owner, name), and the mixer's view is the dict of its entries' views
         self._parts_of: Dict[int, List[str]] = {}
@@ -227,6 +234,7 @@ class SequenceCache:
                 for name, shape, dt in req.tensors:
                     tensors[name] = torch.zeros((self.max_slots, *shape), dtype=dt or dtype, device=self.device)
                 self.states[owner] = StateView(tensors)
+                self.steps_repeatable = self.steps_repeatable and req.repeatable
             else:
                 raise CacheError(f"cache owner {owner}: unknown kind of request {req!r}")
         self.groups: List[KVGroup] = [

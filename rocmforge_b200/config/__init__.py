@@ -6,4 +6,5 @@ from .rifizen import RifizenConfig
 from .vilulorn import VilulornConfig
 from .figalix import FigalixConfig
 from .ludusun import LudusunConfig
+from .gedilorn import GedilornConfig
 from . import vilulorn   # (its builder registers "Vilulorn")

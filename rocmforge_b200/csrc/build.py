@@ -38,6 +38,8 @@ MODULES: Dict[str, List[str]] = {
     "mamba2": ["mamba2.cu", "common.cuh"],
     "mlstm": ["mlstm.cu", "common.cuh"],
     "delta": ["delta.cu", "common.cuh"],
+    "streams": ["streams.cu", "common.cuh"],
+    "latent": ["latent.cu", "common.cuh"],
     "random_fill": ["random_fill.cu", "common.cuh"],
     "gemm_tcgen05": ["gemm_tcgen05.cu", "tcgen05_common.cuh", "common.cuh"],
     # has one CTA load a tile for its whole cluster (this GPU's memory only): a file of its own, left out of
@@ -46,6 +48,8 @@ MODULES: Dict[str, List[str]] = {
     "attention_decode": ["attention_decode.cu", "common.cuh"],
     "attention_prefill": ["attention_prefill.cu", "common.cuh"],
     "attention_prefill_tc": ["attention_prefill_tc.cu", "tcgen05_common.cuh", "common.cuh"],
+    "attention_latent_prefill": ["attention_latent_prefill.cu", "tcgen05_common.cuh", "common.cuh"],
+    "attention_latent_decode": ["attention_latent_decode.cu", "tcgen05_common.cuh", "common.cuh"],
     "attention_decode_noalloc": ["attention_decode_noalloc.cu", "attention_decode_noalloc.h", "attention_decode.cu",
                                  "common.cuh"],
 }

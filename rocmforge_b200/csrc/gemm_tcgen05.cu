@@ -10,8 +10,8 @@
 // few tokens (tiles of up to 64) still streams every weight once with full 128-row MMAs; K may be split
 // across CTAs (grid.z), each split writing its own 32-bit partial sums, which the next
 // add+RMSNorm kernel adds in index order (no atomics: the result never depends on timing).
-// Epilogues: + bias, 32-bit output, accumulate into the 32-bit residual stream, and
-// SwiGLU on row-interleaved gate/up weights.
+// Epilogues: + bias, 32-bit output, accumulate into the 32-bit residual stream, and the
+// units silu(gate) * up (SWIGLU) and relu(gate) * up (REGLU) on row-interleaved gate/up weights.
 //
 // maeddesg/ROCmForge's counterparts are its RDNA-WMMA prefill GEMMs (hip_kernels/wmma/
 // wmma_gemm_tiled.hip:57-195: 64x64x16 tiles, FP16 operands, FP32 accumulate) and its decode
@@ -209,6 +209,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                                 reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.ldo + (n >> 1)] =
                                     __float2bfloat16_rn(silu_fast(g) * u);
                         }
+                    } else if (p.mode == EPI_REGLU) {    // the same exchange, relu instead of silu
+                        const bool odd = lane & 1;
+#pragma unroll
+                        for (int j = 0; j < CH; j += 2) {
+                            const float v0 = __uint_as_float(r[j]) + b, v1 = __uint_as_float(r[j + 1]) + b;
+                            const float got = __shfl_xor_sync(0xffffffffu, odd ? v0 : v1, 1);
+                            const float g = odd ? got : v0, u = odd ? v1 : got;
+                            const int m = m0 + j + (odd ? 1 : 0);
+                            if (m < p.M && (n | 1) < p.N)
+                                reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.ldo + (n >> 1)] = __float2bfloat16_rn(fmaxf(g, 0.f) * u);
+                        }
                     } else if (n < p.N) {
                         // the mode, the output's base and the number of tokens that exist are settled once per chunk: a
                         // token then costs an add and a store (settling them per element made a chunk of 32 tokens take
@@ -366,11 +377,11 @@ extern "C" {
 int rf_gemm_tc_supported(int M, int N, int K, int mode) {
     if (M <= 0 || N <= 0 || K <= 0) return 0;
     if (K % 8) return 0;                              // TMA needs 16-byte row strides
-    if ((mode == EPI_SWIGLU || mode == EPI_CLAMPGLU) && (N % 2)) return 0;
+    if ((mode == EPI_SWIGLU || mode == EPI_CLAMPGLU || mode == EPI_REGLU) && (N % 2)) return 0;
     return encode_fn() != nullptr;
 }
 
-// Tokens as rows: out[M, N] (mode STORE / F32 / RESIDUAL) or out[M, N/2] (SWIGLU).
+// Tokens as rows: out[M, N] (mode STORE / F32 / RESIDUAL) or out[M, N/2] (SWIGLU, REGLU).
 int rf_gemm_tc(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo,
                int M, int N, int K, int mode, int* status, cudaStream_t st) {
     if (!rf_gemm_tc_supported(M, N, K, mode) || mode == EPI_PARTIAL || mode == EPI_RESNORM) return RF_ERR_UNSUPPORTED;

@@ -10,7 +10,7 @@
 #define TC_THREADS 192
 #define TC_WAIT_LIMIT_NS 2000000000ULL      // 2 s
 
-enum { EPI_STORE = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_PARTIAL = 4, EPI_RESNORM = 5, EPI_CLAMPGLU = 6 };
+enum { EPI_STORE = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_PARTIAL = 4, EPI_RESNORM = 5, EPI_CLAMPGLU = 6, EPI_REGLU = 7 };
 
 // What the weights-as-rows kernel needs to finish a residual update and prepare the norm that follows it
 // (mode EPI_RESNORM), and to apply a norm that was prepared that way to its own input (ss_in).
@@ -140,6 +140,66 @@ __device__ __forceinline__ void tcgen05_ld16(uint32_t taddr, uint32_t* r) {
 }
 __device__ __forceinline__ void tcgen05_wait_ld() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
 
+// ---------------------------------------------------------------- what the tcgen05 attention kernels share
+__device__ __forceinline__ float at_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// Weights are rounded to bfloat16 with integer arithmetic (add half an ulp, keep the upper 16 bits): the
+// conversion instruction shares the special-function unit with ex2.  Two variants that measured SLOWER here
+// and were dropped: a share of the exponentials as a polynomial on the FMA pipe (763 -> 734 TFLOP/s at 8,192
+// tokens), and two softmax threads per row (763 -> 435): the softmax warps lack neither ex2 throughput nor
+// threads; what helped was letting the next page's scores be computed while they work (see issue_s).
+__device__ __forceinline__ uint32_t at_pack_bf16x2(float a, float b) {      // a, b >= 0 and finite
+    return __byte_perm(__float_as_uint(a) + 0x8000u, __float_as_uint(b) + 0x8000u, 0x7632);
+}
+
+__device__ __forceinline__ void tcgen05_st32(uint32_t taddr, const uint32_t* r) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
+        "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
+        "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};"
+        ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+          "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]),
+          "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]),
+          "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
+        : "memory");
+}
+__device__ __forceinline__ void tcgen05_st16(uint32_t taddr, const uint32_t* r) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
+        "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
+        ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+          "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+        : "memory");
+}
+// A operand in tensor memory (128 lanes = rows, two bfloat16 per 32-bit column), B through a shared-memory descriptor.
+__device__ __forceinline__ void tcgen05_mma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc,
+                                                    uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+        ::"r"(d_tmem), "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
+}
+__device__ __forceinline__ void tcgen05_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+__device__ __forceinline__ void at_arrive(uint32_t bar) {
+    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
+}
+
+// Descriptor of an MN-major operand tile with the 128-byte swizzle: rows are K (keys), 128 bytes = 64
+// elements of N (head dimensions) per row; 8-row groups 1024 bytes apart (stride byte offset), the next
+// block of 64 N-elements `lbo_bytes` further (leading byte offset).
+__device__ __forceinline__ uint64_t make_smem_desc_mn(uint32_t addr, uint32_t lbo_bytes) {
+    uint64_t d = 0;
+    d |= (uint64_t)((addr & 0x3FFFF) >> 4);
+    d |= (uint64_t)((lbo_bytes >> 4) & 0x3FFF) << 16;
+    d |= (uint64_t)(1024 >> 4) << 32;
+    d |= (uint64_t)1 << 46;
+    d |= (uint64_t)2 << 61;
+    return d;
+}
 // Shared-memory matrix descriptor of a K-major tile whose rows are 128 bytes (64 bf16) wide,
 // written by TMA with the 128-byte swizzle: 8-row groups are 1024 bytes apart.
 __device__ __forceinline__ uint64_t make_smem_desc(uint32_t addr) {
@@ -212,6 +272,25 @@ template <int CH>
 __device__ __forceinline__ void epilogue_rows(const TcParams& p, const uint32_t* r, int m, int n0) {
     if (m >= p.M) return;
     const bool whole = n0 + CH <= p.N;
+    if (p.mode == EPI_REGLU) {                       // relu(gate) * up on row-interleaved gate/up columns
+        __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)m * p.ldo + (n0 >> 1);
+        if (whole && !(reinterpret_cast<uintptr_t>(o) & 15)) {
+#pragma unroll
+            for (int j = 0; j < CH; j += 16) {
+                uint32_t w[4];
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+                    w[q] = pack_bf16x2(fmaxf(__uint_as_float(r[j + 4 * q]), 0.f) * __uint_as_float(r[j + 4 * q + 1]),
+                                       fmaxf(__uint_as_float(r[j + 4 * q + 2]), 0.f) * __uint_as_float(r[j + 4 * q + 3]));
+                *reinterpret_cast<uint4*>(o + (j >> 1)) = make_uint4(w[0], w[1], w[2], w[3]);
+            }
+            return;
+        }
+#pragma unroll
+        for (int j = 0; j < CH; j += 2)
+            if (n0 + j + 1 < p.N) o[j >> 1] = __float2bfloat16_rn(fmaxf(__uint_as_float(r[j]), 0.f) * __uint_as_float(r[j + 1]));
+        return;
+    }
     if (p.mode == EPI_SWIGLU) {
         __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)m * p.ldo + (n0 >> 1);
         if (whole && !(reinterpret_cast<uintptr_t>(o) & 15)) {

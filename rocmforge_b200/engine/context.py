@@ -86,6 +86,23 @@ class StepContext:
             return tc.gemm_tc(x, w, bias, mode=mode)
         return kernels.gemm_simt(x, w, bias, out_f32=out_f32)
 
+    def matmul_rows_or_parts(self, x, w):
+        """x w^T as [M, N] in the compute dtype, or, where few tokens let K be split, as the float32 stack [S, M, N] of partial
+        sums (for consumers that add them up themselves)."""
+        tc = kernels.tensor_core
+        if isinstance(x, ScaledRows):
+            x = x.materialize()
+        if x.shape[0] <= tc.SKINNY_MAX_TOKENS:
+            if self.uses_tensor_cores(x, w, tc.PARTIAL):
+                splits = tc.split_k_for(w.shape[0], w.shape[1], tokens=x.shape[0])
+                if splits > 1:
+                    return tc.gemm_tc_skinny(x, w, mode=tc.PARTIAL, splits=splits)
+            elif not self.uses_tensor_cores(x, w, tc.STORE):
+                splits = kernels.split_k_for_simt(w.shape[0], w.shape[1])
+                if splits > 1:
+                    return kernels.gemm_simt(x, w, splits=splits)
+        return self.matmul(x, w)
+
     def matmul_f32_parts(self, x, w):
         """x w^T as float32 [M, N], or for few tokens as the stack [S, M, N] of a K-split product's partial sums (the
         number of splits follows the weight's shape and the step's token bucket, never the batch's content)."""
@@ -139,16 +156,17 @@ class StepContext:
         stream.flush()
         kernels.gemm_simt(x, w, bias, out=stream.h, accumulate=True)
 
-    def gated_activation(self, y, gate_up):
-        """silu(gate) * up from the fused, row-interleaved gate/up matrix."""
+    def gated_activation(self, y, gate_up, activation: str = "silu"):
+        """silu(gate) * up (or relu(gate) * up) from the fused, row-interleaved gate/up matrix."""
         tc = kernels.tensor_core
         w = gate_up.weight
-        y, row_ss = self.unpack_rows(y, w, tc.SWIGLU)
-        if gate_up.bias is None and self.uses_tensor_cores(y, w, tc.SWIGLU):
+        mode = {"silu": tc.SWIGLU, "relu": tc.REGLU}[activation]
+        y, row_ss = self.unpack_rows(y, w, mode)
+        if gate_up.bias is None and self.uses_tensor_cores(y, w, mode):
             if y.shape[0] <= tc.SKINNY_MAX_TOKENS:
-                return tc.gemm_tc_skinny(y, w, mode=tc.SWIGLU, row_ss=row_ss)
-            return tc.gemm_tc(y, w, mode=tc.SWIGLU)
+                return tc.gemm_tc_skinny(y, w, mode=mode, row_ss=row_ss)
+            return tc.gemm_tc(y, w, mode=mode)
         if row_ss is not None:
             y = ScaledRows(y, row_ss[0], row_ss[1], w.shape[1]).materialize()
         gu = self.matmul(y, w, gate_up.bias)
-        return kernels.swiglu(gu)
+        return kernels.swiglu(gu, activation=activation)

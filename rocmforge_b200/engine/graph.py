@@ -315,9 +315,9 @@ class DecodeRunner:
         else:
             self.launched_ahead += 1
         cache.commit(slots, [1] * B)                       # the step is under way for these sequences
-        if more and not cache.states:
+        if more and cache.steps_repeatable:
             # (a model with per-sequence state is not run ahead: a step that is dropped would have changed the state,
-            # whereas keys and values written by a dropped step are simply written again)
+            # whereas keys and values written by a dropped step, and state kept for that, are simply written again)
             # the next step of the same sequences, before the host knows this step's ids
             try:
                 cache.prepare(slots, [1] * B)

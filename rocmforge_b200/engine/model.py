@@ -25,6 +25,9 @@ from .context import Options, StepContext
 from .stream import ResidualStream
 
 
+EMBEDDING = -1          # the embedding's place among the cache's owners (the others are schedule indices)
+
+
 @dataclass
 class ScheduleEntry:
     """One execution of a layer.  ``kv_from``: index of an earlier schedule entry whose cache
@@ -54,6 +57,7 @@ class ModelSpec:
     pass_offsets_prefix: str = ""
     positions: Optional[Part] = None                 # parts.embedding.LearnedPositions: a learned vector per position, added to the embedding
     positions_prefix: str = ""
+    streams: Optional[int] = None                    # several residual streams (parts.streams): ``stream.h`` is then [T, streams, width]
 
     def named_parts(self) -> Dict[str, Part]:
         """{tensor-name prefix: leaf part}."""
@@ -77,8 +81,10 @@ class ModelSpec:
         return out
 
     def cache_requests(self) -> Dict[int, object]:
-        """{schedule index: what that execution's mixer keeps per sequence}."""
+        """{schedule index: what that execution's mixer keeps per sequence; EMBEDDING: what the embedding keeps}."""
         out = {}
+        if hasattr(self.embedding, "cache_request"):
+            out[EMBEDDING] = self.embedding.cache_request()
         for i, e in enumerate(self.schedule):
             if not 0 <= e.layer < len(self.blocks):
                 raise ValueError(f"schedule entry {i} names layer {e.layer}; there are {len(self.blocks)}")
@@ -204,8 +210,12 @@ class Model:
             stream = ResidualStream(h)
             if y is not None:
                 stream.prepared = (first, y)
+        elif hasattr(spec.embedding, "cache_request"):
+            stream = ResidualStream(spec.embedding.forward(ctx, ctx.tokens, cache.view(EMBEDDING)))
         else:
             stream = ResidualStream(spec.embedding.forward(ctx, ctx.tokens))
+        if spec.streams is not None:
+            stream.h = stream.h[:, None]             # all streams equal: one row stands for all until the first update
         if spec.schedule and spec.schedule[0].pass_index is not None:
             spec.pass_offsets.add(ctx, stream, spec.schedule[0].pass_index)
         for i, entry in enumerate(spec.schedule):

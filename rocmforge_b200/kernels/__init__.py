@@ -9,5 +9,7 @@ from .basic import (relu2, add_row, branch_norm_add, head_norm_kv_write, gemm_si
 from .basic import (embed_positions, round_rows, clamped_glu, sigmoid_gate, key_span, gla_prepare, gla_scan, MOE_SCORINGS)
 from .basic import (dyt_rows, scaled_add, softcap_, gated_scan, gated_chunked, mlstm_prepare, mlstm_gates, conv_silu, mamba_gates, mamba_finish)
 from .basic import (weighted_add, stretch_norm, delta_prepare, delta_scan)
+from .latent import (streams_update, pair_embed, scale_, latent_write, latent_gather, head_product, attention_latent_prefill,
+                     attention_latent_prefill_supported, attention_latent_decode, attention_latent_decode_groups)
 from ._ffi import launch_count
 from . import tensor_core

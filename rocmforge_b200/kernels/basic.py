@@ -201,14 +201,15 @@ def rope_kv_write(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: in
     return q_out
 
 
-def swiglu(gu: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
-    """a[t, j] = silu(gu[t, 2j]) * gu[t, 2j+1]."""
+def swiglu(gu: torch.Tensor, out: torch.Tensor | None = None, activation: str = "silu") -> torch.Tensor:
+    """a[t, j] = silu(gu[t, 2j]) * gu[t, 2j+1] (``activation`` "relu": relu instead of silu)."""
+    need(activation in ("silu", "relu"), f"swiglu: activation {activation!r} (silu, relu)")
     need_cuda(gu)
     need(gu.dim() == 2 and gu.is_contiguous() and gu.shape[1] % 2 == 0, "swiglu: input must be [T, 2I]")
     T, I2 = gu.shape
     if out is None:
         out = torch.empty((T, I2 // 2), dtype=gu.dtype, device=gu.device)
-    f = _f("elementwise", "rf_swiglu", c_int, c_void_p, c_void_p, c_int, c_int, c_void_p)
+    f = _f("elementwise", "rf_swiglu" if activation == "silu" else "rf_reglu", c_int, c_void_p, c_void_p, c_int, c_int, c_void_p)
     check(f(dtype_code(gu.dtype), ptr(gu), ptr(out), T, I2 // 2, stream()), "swiglu")
     return out
 
@@ -288,11 +289,24 @@ def attention_generic(q: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: 
     need(q.dim() == 2 and q.stride(1) == 1, "attention: q must be [T, >= heads*head_dim] with unit inner stride")
     need(k_pages.dtype == q.dtype and v_pages.dtype == q.dtype, "attention: cache dtype differs from q")
     need(tuple(k_pages.shape[1:]) == (n_kv_heads, PAGE, head_dim) and k_pages.is_contiguous()
-         and tuple(v_pages.shape) == (k_pages.shape[0], n_kv_heads, PAGE, vd) and v_pages.is_contiguous(),
+         and tuple(v_pages.shape) == (k_pages.shape[0], n_kv_heads, PAGE, vd)
+         and (v_pages.is_contiguous() or v_pages.stride() == k_pages.stride()),
          "attention: bad cache page shape")
     if out is None:
         out = torch.empty((T, n_heads * vd), dtype=q.dtype, device=q.device)
     window = key_span(window, chunk)
+    if not v_pages.is_contiguous():
+        # values that are the first vd numbers of the key rows
+        need(not softcap and slopes is None and not keep_first and sinks is None,
+             "attention: values inside key rows go with a plain softmax only")
+        f = _f("attention_generic", "rf_attention_generic_rows", c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
+               c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
+               c_void_p)
+        check(f(dtype_code(q.dtype), ptr(q), q.stride(0), ptr(out), out.stride(0), ptr(k_pages), ptr(v_pages), head_dim,
+                ptr(tok_seq), ptr(tok_pos), ptr(seq_slot), ptr(block_table), block_table.shape[1], n_heads, n_kv_heads,
+                head_dim, vd, float(scale), window, T, stream()),
+              f"attention_generic (heads={n_heads}, kv_heads={n_kv_heads}, head_dim={head_dim}, values in {vd} of them)")
+        return out
     keep_first = int(keep_first or 0) if window > 0 else 0         # without a window every key is visible anyway
     if sinks is not None:
         need_cuda(sinks)

@@ -8,7 +8,8 @@ import torch
 
 from ._ffi import KernelError, sm_count as device_sm_count, c_float, c_int, c_ll, c_void_p, check, fn, need, need_cuda, ptr, stream
 
-STORE, F32, RESIDUAL, SWIGLU, PARTIAL, RESNORM, CLAMPGLU = 0, 1, 2, 3, 4, 5, 6
+STORE, F32, RESIDUAL, SWIGLU, PARTIAL, RESNORM, CLAMPGLU, REGLU = 0, 1, 2, 3, 4, 5, 6, 7
+GATED = (SWIGLU, REGLU)      # modes whose output is half as wide as the (row-interleaved) weight
 SKINNY_MAX_TOKENS = 128     # above it the large-M kernels stream the weights better (7B shape, decode step: 128 tokens
                             # 5.09 ms skinny / 6.38 ms clustered; 192 tokens as tiles of 64: 7.78 / 6.73)
 
@@ -131,14 +132,14 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = Non
             out: Optional[torch.Tensor] = None, cluster: Optional[int] = None,
             parts: int = 0) -> torch.Tensor:
     """Tokens as accumulator rows (any M).  STORE -> bf16 [M,N]; F32 -> f32 [M,N]; RESIDUAL: out (f32) += x w^T;
-    SWIGLU -> bf16 [M, N/2] from row-interleaved gate/up weights.  ``parts`` (clustered kernel, RESIDUAL only):
+    SWIGLU / REGLU -> bf16 [M, N/2] = silu / relu (gate) * up from row-interleaved gate/up weights.  ``parts`` (clustered kernel, RESIDUAL only):
     K parts whose sums are added one after the other, 0 = the kernel's own choice."""
     _common(x, w, bias, out)
     M, K = x.shape
     N = w.shape[0]
     need(supported(M, N, K, mode), f"tensor-core gemm: shape {M}x{N}x{K} is not supported")
-    cols = N // 2 if mode == SWIGLU else N
-    odt = torch.bfloat16 if mode in (STORE, SWIGLU) else torch.float32
+    cols = N // 2 if mode in GATED else N
+    odt = torch.bfloat16 if mode == STORE or mode in GATED else torch.float32
     if out is None:
         need(mode != RESIDUAL, "gemm: RESIDUAL needs the tensor to add into")
         out = torch.empty((M, cols), dtype=odt, device=x.device)
@@ -251,8 +252,8 @@ def gemm_tc_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor
     need(supported(M, N, K, mode), f"tensor-core gemm: shape {M}x{N}x{K} is not supported")
     need(mode != RESNORM, "skinny gemm: the fused residual + norm epilogue has its own function")
     need(splits == 1 or mode == PARTIAL, "skinny gemm: several K splits need mode PARTIAL")
-    cols = N // 2 if mode == SWIGLU else N
-    odt = torch.bfloat16 if mode in (STORE, SWIGLU) else torch.float32
+    cols = N // 2 if mode in GATED else N
+    odt = torch.bfloat16 if mode == STORE or mode in GATED else torch.float32
     shape = (splits, M, N) if mode == PARTIAL else (M, cols)
     if out is None:
         need(mode != RESIDUAL, "gemm: RESIDUAL needs the tensor to add into")

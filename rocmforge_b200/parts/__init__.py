@@ -22,5 +22,7 @@ from .block import ScaledPreNormBlock
 from .mlp import SummedFeedForward
 from .mlstm import MatrixMemory
 from .mamba2 import StateSpaceDuality
-from .latent import LatentAttention
+from .latent import LatentAttention, LatentCacheAttention
 from .delta import GatedDeltaRule
+from .embedding import PairEmbedding
+from .streams import HyperConnectedBlock, HyperConnection, StreamsNorm

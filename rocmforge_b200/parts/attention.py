@@ -15,6 +15,16 @@ from .base import MIXERS, Mixer, POSITIONS
 from .linear import Linear
 
 
+def query_tiles(batch, rows: int) -> np.ndarray:
+    """(sequence, first row) pairs of the step's query tiles of ``rows`` rows, by the keys a tile sees (none for steps of one token
+    per sequence)."""
+    if batch.is_decode:
+        return np.zeros((0,), dtype=np.int32)
+    tiles = [(i, q0) for i in range(batch.B) for q0 in range(0, int(batch.n_new[i]), rows)]
+    tiles.sort(key=lambda t: int(batch.starts[t[0]]) + t[1])
+    return np.asarray(tiles, dtype=np.int32).reshape(-1)
+
+
 @MIXERS.register("gqa_attention")
 class GQAAttention(Mixer):
     """q/k/v projections (with or without bias), rotation of q and k, write of k and v into
@@ -216,12 +226,7 @@ class GQAAttention(Mixer):
         """(sequence, first row) of every query tile of the step's new tokens, sorted by the keys a tile sees (the
         kernels start with the heaviest): decided on the host so that the device never searches.  Steps of one token
         per sequence need none."""
-        if batch.is_decode:
-            return np.zeros((0,), dtype=np.int32)
-        rows = self.TILE_ROWS[name]
-        tiles = [(i, q0) for i in range(batch.B) for q0 in range(0, int(batch.n_new[i]), rows)]
-        tiles.sort(key=lambda t: int(batch.starts[t[0]]) + t[1])
-        return np.asarray(tiles, dtype=np.int32).reshape(-1)
+        return query_tiles(batch, self.TILE_ROWS[name])
 
     def forward(self, ctx, y, cache_view, stream):
         self.o.add_to_stream(ctx, self.heads_out(ctx, y, cache_view), stream)

@@ -13,7 +13,7 @@ from .linear import Linear
 
 @FEED_FORWARDS.register("gated_mlp")
 class GatedMLP(FeedForward):
-    """x += W_down (act(W_gate y) * (W_up y)), no biases
+    """x += W_down (act(W_gate y) * (W_up y)), no biases, act = silu (``activation`` "relu": relu)
     (maeddesg/ROCmForge src/gpu/forward.rs:1094-1161, hip_kernels/elementwise.hip:72-82).
 
     gate and up are fused into one matrix at load time with their rows interleaved
@@ -26,9 +26,9 @@ class GatedMLP(FeedForward):
 
     def __init__(self, hidden: int, intermediate: int, activation: str = "silu", names: Optional[Dict[str, str]] = None):
         """``names``: the tensors' names below the part's prefix (keys gate, up, down)."""
-        if activation != "silu":
+        if activation not in ("silu", "relu"):
             raise ValueError(f"gated_mlp: activation {activation!r} has no kernel")
-        self.hidden, self.intermediate = hidden, intermediate
+        self.hidden, self.intermediate, self.activation = hidden, intermediate, activation
         self.names = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
         self.names.update(names or {})
         self.gate_up: Optional[Linear] = None
@@ -51,11 +51,11 @@ class GatedMLP(FeedForward):
         return ["elementwise"]
 
     def forward(self, ctx, y, stream):
-        a = ctx.gated_activation(y, self.gate_up)                           # [T, I]
+        a = ctx.gated_activation(y, self.gate_up, self.activation)          # [T, I]
         self.down.add_to_stream(ctx, a, stream)
 
     def output(self, ctx, y):
-        return self.down.f32_parts(ctx, ctx.gated_activation(y, self.gate_up))
+        return self.down.f32_parts(ctx, ctx.gated_activation(y, self.gate_up, self.activation))
 
 
 @FEED_FORWARDS.register("relu2_mlp")
