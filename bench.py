@@ -496,6 +496,26 @@ def ludusun_shape(width, layers=4):
     return lud, fig
 
 
+def gedilorn_shape(width, layers=4):
+    """A Gedilorn configuration with layers of the size a real model has: heads of 128 unrotated and 64 rotated dimensions with
+    stretched frequencies and values of 128, a latent of 512 (a cache row of 576 numbers for all heads), without and with the
+    output gate in turn, four residual streams, a dense feed-forward of 4 x width, a table of 32,749 pairs.  And a Ludusun
+    configuration of equal width, heads and depth whose layers are all its latent attention (its closest relative here: keys and
+    values expanded from a latent of 512, queries from one of width / 2, all earlier positions visible), with the same
+    feed-forward."""
+    heads = width // 128
+    rot = dict(dims=64, base=1e6, scaling=dict(factor=8.0, original=8192, fast=32.0, slow=1.0))
+    mix = dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot=rot)
+    dense = dict(kind="dense", ff=4 * width)
+    ged = dict(architecture="Gedilorn", vocab=32000, width=width, norm=dict(eps=1e-6), streams=4, logit_scale=0.5,
+               embedding=dict(scale=2.0, bigram=dict(buckets=32749, mul_prev=7919, mul_cur=104729)),
+               layers=[dict(type=("latent_attention", "latent_attention_2")[i % 2], mixer=mix, mlp=dense) for i in range(layers)])
+    lat = dict(heads=heads, dim=128, vdim=128, q_rank=width // 2, kv_rank=512, scale=128 ** -0.5)
+    lud = dict(architecture="Ludusun", vocab=32000, width=width, norm=dict(eps=1e-6), embedding=dict(scale=2.0), logit_softcap=30.0,
+               layers=[dict(type="latent_attention", mixer=lat, mlp=dense) for _ in range(layers)])
+    return ged, lud
+
+
 def rifizen_points(pk, seed, widths=(1024, 2048), tokens=PREFILL_TOKENS, batches=(8, 64), steps=64, warmup=8,
                    names=("rifizen", "dense"), archs=("Rifizen", "Qwen2ForCausalLM"), shapes=None):
     """Prefill and decode of one design at layer sizes of a real model, beside another at equal size (by default Rifizen
@@ -609,7 +629,7 @@ def main():
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the configuration (named in config)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (quick check)")
-    ap.add_argument("--only", choices=["decode", "prefill", "ablate", "0.5b", "14b", "rifizen", "vilulorn", "figalix", "ludusun"], default=None,
+    ap.add_argument("--only", choices=["decode", "prefill", "ablate", "0.5b", "14b", "rifizen", "vilulorn", "figalix", "ludusun", "gedilorn"], default=None,
                     help="run one phase only and print a short line (small cases for profilers)")
     ap.add_argument("--shape", choices=["7b", "0.5b", "14b"], default="7b",
                     help="layer sizes for --only decode / prefill / ablate (the full run always measures all three)")
@@ -649,6 +669,12 @@ def main():
                           "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops") if k in pk},
                           **rifizen_points(pk, args.seed, steps=min(args.steps, 64), warmup=warmup, names=("figalix", "rifizen"),
                                            archs=("Figalix", "Rifizen"), shapes=figalix_shape)}))
+        return 0
+    if args.only == "gedilorn":
+        print(json.dumps({"only": "gedilorn", "tokens": PREFILL_TOKENS, "prompt_len": PROMPT_LEN,
+                          "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops") if k in pk},
+                          **rifizen_points(pk, args.seed, steps=min(args.steps, 64), warmup=warmup, names=("gedilorn", "ludusun"),
+                                           archs=("Gedilorn", "Ludusun"), shapes=gedilorn_shape)}))
         return 0
     if args.only == "ludusun":
         print(json.dumps({"only": "ludusun", "tokens": PREFILL_TOKENS, "prompt_len": PROMPT_LEN,

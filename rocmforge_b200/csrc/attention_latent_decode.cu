@@ -11,9 +11,9 @@
 //                                            weights, written to shared memory by the softmax warps
 // so a page comes into shared memory once (TMA, 128-byte swizzle, two or more stages) and is used for both.
 // A CTA owns (token, group of heads) and every splits-th page; the CTAs of a token are a thread-block cluster and merge
-// their (maximum, sum, O) through distributed shared memory: no scratch memory, no atomics.
+// their (reference, sum, O) through distributed shared memory: no scratch memory, no atomics.
 //   warp 0  TMA producer (pages older than the step are asked for before the dependency wait)
-//   warp 1  issues the MMAs; the scores of the next page are computed under the softmax of this one
+//   warp 1  issues the MMAs, scores up to two pages ahead of the softmax
 //   warps 2-5  softmax: the 64 rows of an M = 64 accumulator lie in the first 16 lanes of each 32-lane quarter of tensor
 //           memory, so a lane below 16 owns one key and all heads.  The exponentials' reference of a head moves only when
 //           some score exceeds it by more than 8 (log2 units): one vote a page instead of a maximum a head; sums of weights
@@ -47,12 +47,12 @@ __device__ __forceinline__ uint32_t ld_peer(uint32_t addr, int rank) {
     asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
     return r;
 }
-__device__ __forceinline__ float ld_remote(uint32_t addr) {
-    float v;
-    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+__device__ __forceinline__ float2 ld_pull2(uint32_t addr) {
+    float2 v;
+    asm volatile("ld.shared::cluster.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(addr) : "memory");
     return v;
 }
-__device__ __forceinline__ float4 ld_remote4(uint32_t addr) {
+__device__ __forceinline__ float4 ld_pull4(uint32_t addr) {
     float4 v;
     asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
     return v;
@@ -65,6 +65,29 @@ __device__ __forceinline__ bool ld_group_any(bool mine) {        // whether any 
                  "barrier.cta.red.or.pred p, 1, 128, q;\n\t"
                  "selp.u32 %0, 1, 0, p;\n\t}" : "=r"(any) : "r"((uint32_t)mine) : "memory");
     return any != 0;
+}
+// Whether the phase of parity `parity` is over; never suspends the thread.
+__device__ __forceinline__ bool ld_test(uint32_t bar, uint32_t parity) {
+    uint32_t ok;
+    asm volatile("{\n\t.reg .pred p;\n\t"
+                 "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+                 "selp.u32 %0, 1, 0, p;\n\t}" : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
+    return ok != 0;
+}
+// Over the 16 lanes of each half warp: lane l ends with op(v[l % 16] of all of them); 15 exchanges instead of 16 x 4.
+template <bool MAX>
+__device__ __forceinline__ float ld_scatter16(float* v, int lane) {
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) {
+        const bool up = lane & o;
+#pragma unroll
+        for (int j = 0; j < o; ++j) {
+            const float send = up ? v[j] : v[j + o], keep = up ? v[j + o] : v[j];
+            const float got = __shfl_xor_sync(0xffffffffu, send, o);
+            v[j] = MAX ? fmaxf(keep, got) : keep + got;
+        }
+    }
+    return v[0];
 }
 // bf16 x bf16 -> f32; a_mn: A is MN-major
 __device__ __forceinline__ uint32_t ld_idesc(int m, int n, int a_mn) {
@@ -80,11 +103,11 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
     uint8_t* q_s = c_s + (size_t)a.stages * tile_bytes;            // [nb][NH][128 B]
     uint8_t* p_s = q_s + (size_t)a.nb * NH * 128;                  // [2][NH][128 B]
     float* m_s = reinterpret_cast<float*>(p_s + 2 * NH * 128);     // [NH] the heads' references (log2 units)
-    float* l_s = m_s + NH;                                         // [NH] the heads' sums
-    float* corr_s = l_s + NH;                                      // [NH]
+    float* l_s = m_s + NH;                                         // [NH][2] the heads' references and sums, for the merge
+    float* corr_s = l_s + 2 * NH;                                      // [NH]
     float* part_s = corr_s + NH;                                   // [4][NH] per-warp maxima, then sums
-    float* wts_s = part_s + 4 * NH;                                // [LD_MAX_SPLITS][NH]
-    uint64_t* bars = reinterpret_cast<uint64_t*>(wts_s + LD_MAX_SPLITS * NH);
+    float* wts_s = part_s + 4 * NH;                                // [LD_MAX_SPLITS][NH][2] the merge: references (then weights) and sums
+    uint64_t* bars = reinterpret_cast<uint64_t*>(wts_s + 2 * LD_MAX_SPLITS * NH);
     // q_full, s_full[2], p_ready[2], pv_done[2] (two each: no barrier completes two phases between two looks of a waiter),
     // c_full[4], c_free[4]
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
@@ -114,7 +137,7 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
         tcgen05_alloc(smem_u32(tmem_slot), a.tmem_cols);
         tcgen05_relinquish();
     }
-    if (threadIdx.x >= 64 && threadIdx.x - 64 < NH) { m_s[threadIdx.x - 64] = -INFINITY; l_s[threadIdx.x - 64] = 0.f; }
+    if (threadIdx.x >= 64 && threadIdx.x - 64 < NH) { m_s[threadIdx.x - 64] = -INFINITY; }
     tcgen05_fence_before();
     __syncthreads();
     tcgen05_fence_after();
@@ -145,38 +168,46 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
             for (; ok && i < n_t; ++i) ok = load(i);
         }
     } else if (warp == 1) {
-        if (lane == 0) {
+        if (elect_one()) {
             const uint32_t idesc_s = ld_idesc(64, NH, 0), idesc_o = ld_idesc(128, NH, 1);
-            auto issue_s = [&](int i) -> bool {
-                const int st = i % a.stages;
-                if (!mbar_wait(b_cfull + 8 * st, (i / a.stages) & 1, &abort_flag)) return false;
-                tcgen05_fence_after();
-                const uint32_t c_t = smem_u32(c_s) + st * tile_bytes, q_t = smem_u32(q_s), d = tmem_s + (i & 1) * NH;
-                for (int ks = 0; ks < a.n_steps; ++ks)
-                    tcgen05_mma_bf16(d, make_smem_desc(c_t + (ks >> 2) * LD_PAGE_BLOCK + (ks & 3) * 32),
-                                     make_smem_desc(q_t + (ks >> 2) * NH * 128 + (ks & 3) * 32), idesc_s, ks ? 1u : 0u);
-                tcgen05_commit(b_sfull + 8 * (i & 1));
-                return true;
-            };
             bool ok = mbar_wait(b_q, 0, &abort_flag);              // (also with no page of its own: the copy must have landed)
-            if (ok && n_t > 0) ok = issue_s(0);
-            for (int i = 0; i < n_t && ok; ++i) {
-                const int st = i % a.stages;
-                // one stage only: the next page cannot arrive before this one's values are used
-                if (a.stages > 1 && i + 1 < n_t) { ok = issue_s(i + 1); if (!ok) break; }
-                ok = mbar_wait(b_pready + 8 * (i & 1), (i >> 1) & 1, &abort_flag);
-                if (!ok) break;
-                tcgen05_fence_after();
-                const int cnt = min(RF_PAGE, pos + 1 - (p_lo + i * a.splits) * RF_PAGE);
-                const int k_steps = (cnt + 15) >> 4;               // 16 keys each; rows behind the last key are zeroed up to there
-                const uint32_t c_t = smem_u32(c_s) + st * tile_bytes, p_t = smem_u32(p_s) + (i & 1) * NH * 128;
-                for (int mb = 0; mb < a.m_blocks; ++mb)
-                    for (int ks = 0; ks < k_steps; ++ks)
-                        tcgen05_mma_bf16(tmem_o + mb * NH, make_smem_desc_mn(c_t + 2 * mb * LD_PAGE_BLOCK + ks * 16 * 128, LD_PAGE_BLOCK),
-                                         make_smem_desc(p_t + ks * 32), idesc_o, (i | ks) ? 1u : 0u);
-                tcgen05_commit(b_cfree + 8 * st);
-                tcgen05_commit(b_pvdone + 8 * (i & 1));
-                if (a.stages == 1 && i + 1 < n_t) ok = issue_s(i + 1);
+            // Two kinds of work, each in page order: the scores of page si (its copy has landed, the softmax has read the scores of
+            // page si - 2) and the values of page vi (its weights are written).  Values first: they free a place in the ring.
+            // Neither waits behind the other: waiting for page si's copy with page vi's weights at hand would hold up the very copy.
+            int si = 0, vi = 0;
+            unsigned long long t0 = 0;
+            for (int spin = 0; ok && vi < n_t; ++spin) {
+                if (vi < si && ld_test(b_pready + 8 * (vi & 1), (vi >> 1) & 1)) {
+                    tcgen05_fence_after();
+                    const int cnt = min(RF_PAGE, pos + 1 - (p_lo + vi * a.splits) * RF_PAGE), st = vi % a.stages;
+                    const int k_steps = (cnt + 15) >> 4;           // 16 keys each; rows behind the last key are zeroed up to there
+                    uint64_t cd = make_smem_desc_mn(smem_u32(c_s) + st * tile_bytes, LD_PAGE_BLOCK);
+                    const uint64_t pd = make_smem_desc(smem_u32(p_s) + (vi & 1) * NH * 128);
+                    for (int mb = 0; mb < a.m_blocks; ++mb, cd += (2 * LD_PAGE_BLOCK) >> 4)
+#pragma unroll
+                        for (int ks = 0; ks < 4; ++ks)              // 16 keys = 16 rows of 128 bytes further in C, 32 bytes in P
+                            if (ks < k_steps) tcgen05_mma_bf16(tmem_o + mb * NH, cd + ks * (16 * 128 >> 4), pd + 2 * ks, idesc_o, (vi | ks) ? 1u : 0u);
+                    tcgen05_commit(b_cfree + 8 * st);
+                    tcgen05_commit(b_pvdone + 8 * (vi & 1));
+                    ++vi;
+                    spin = 0; t0 = 0;
+                } else if (si < n_t && si < vi + 2 && ld_test(b_cfull + 8 * (si % a.stages), (si / a.stages) & 1)) {
+                    tcgen05_fence_after();
+                    uint64_t cd = make_smem_desc(smem_u32(c_s) + (si % a.stages) * tile_bytes), qd = make_smem_desc(smem_u32(q_s));
+                    const uint32_t d = tmem_s + (si & 1) * NH;
+                    for (int b = 0; b < a.nb; ++b, cd += LD_PAGE_BLOCK >> 4, qd += (NH * 128) >> 4)
+#pragma unroll
+                        for (int k = 0; k < 4; ++k)
+                            if (4 * b + k < a.n_steps) tcgen05_mma_bf16(d, cd + 2 * k, qd + 2 * k, idesc_s, (b | k) ? 1u : 0u);
+                    tcgen05_commit(b_sfull + 8 * (si & 1));
+                    ++si;
+                    spin = 0; t0 = 0;
+                } else if ((spin & 63) == 63) {                    // bounded, like every wait here
+                    if (*(volatile int*)&abort_flag) ok = false;
+                    const unsigned long long now = global_ns();
+                    if (t0 == 0) t0 = now;
+                    if (now - t0 > TC_WAIT_LIMIT_NS) { abort_flag = 1; ok = false; }
+                }
             }
         }
     } else {
@@ -185,9 +216,11 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
         const int my_row = quarter * 16 + lane;                    // of the page, for lanes below 16
         const float sl2 = a.scale * 1.4426950408889634f;
         const uint32_t p_chunk = (uint32_t)(my_row >> 3), p_byte = (uint32_t)(my_row & 7) * 2;
-        float l[NH];
+        constexpr bool REG = NH <= 32;                             // the heads' references also in registers
+        float l[NH], m_reg[REG ? NH : 1];
 #pragma unroll
-        for (int h = 0; h < NH; ++h) l[h] = 0.f;
+        for (int h = 0; h < NH; ++h) { l[h] = 0.f; if (REG) m_reg[h] = -INFINITY; }
+        auto ref = [&](int h) { return REG ? m_reg[REG ? h : 0] : m_s[h]; };
         pdl_wait();                                                // the output may still be read by a kernel before us
         bool ok = true;
         for (int i = 0; i < n_t; ++i) {
@@ -222,15 +255,18 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
 #pragma unroll
             for (int h = 0; h < NH; ++h) {
                 s[h] = visible ? s[h] * sl2 : -INFINITY;
-                moves |= s[h] > m_s[h] + 8.f;
+                moves |= s[h] > ref(h) + 8.f;
             }
             bool seen = i == 0;                                    // whether this step has looked at the previous P V's barrier
             if (ld_group_any(moves)) {
                 if (ld_group_any(!ok)) { ok = false; break; }      // somebody gave up: all leave together
 #pragma unroll
-                for (int h = 0; h < NH; ++h) {
-                    const float w = warp_max(s[h]);
-                    if (lane == 0) part_s[quarter * NH + h] = w;
+                for (int c0 = 0; c0 < NH; c0 += 16) {
+                    float v[16];
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) v[j] = s[c0 + j];
+                    const float w = ld_scatter16<true>(v, lane);   // (the upper half warp holds no keys)
+                    if (lane < 16) part_s[quarter * NH + c0 + lane] = w;
                 }
                 ld_group_sync();
                 if (tid < NH) {
@@ -241,7 +277,7 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
                 }
                 ld_group_sync();
 #pragma unroll
-                for (int h = 0; h < NH; ++h) l[h] *= corr_s[h];
+                for (int h = 0; h < NH; ++h) { l[h] *= corr_s[h]; if (REG) m_reg[h] = m_s[h]; }
                 if (i > 0) {
                     ok = mbar_wait(b_pvdone + 8 * ((i - 1) & 1), ((i - 1) >> 1) & 1, &abort_flag);
                     seen = true;
@@ -265,7 +301,7 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
                 const uint32_t p_t = smem_u32(p_s) + (i & 1) * NH * 128 + p_byte;
 #pragma unroll
                 for (int h = 0; h < NH; ++h) {
-                    const float p = at_exp2(s[h] - m_s[h]);
+                    const float p = at_exp2(s[h] - ref(h));
                     l[h] += p;
                     const unsigned short b = __bfloat16_as_ushort(__float2bfloat16_rn(p));
                     asm volatile("st.shared.u16 [%0], %1;" ::"r"(p_t + h * 128 + ((p_chunk ^ (h & 7)) << 4)), "h"(b) : "memory");
@@ -282,34 +318,52 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
         if (ok && n_t > 0) ok = mbar_wait(b_pvdone + 8 * ((n_t - 1) & 1), ((n_t - 1) >> 1) & 1, &abort_flag);
         // sums over the keys
 #pragma unroll
-        for (int h = 0; h < NH; ++h) {
-            const float w = warp_sum(l[h]);
-            if (lane == 0) part_s[quarter * NH + h] = w;
+        for (int c0 = 0; c0 < NH; c0 += 16) {
+            const float w = ld_scatter16<false>(l + c0, lane);
+            if (lane < 16) part_s[quarter * NH + c0 + lane] = w;
         }
         ld_group_sync();
-        if (tid < NH) l_s[tid] = (part_s[tid] + part_s[NH + tid]) + (part_s[2 * NH + tid] + part_s[3 * NH + tid]);
+        if (tid < NH) {
+            const float sum = (part_s[tid] + part_s[NH + tid]) + (part_s[2 * NH + tid] + part_s[3 * NH + tid]);
+            *reinterpret_cast<float2*>(l_s + 2 * tid) = make_float2(m_s[tid], sum);
+            corr_s[tid] = sum > 0.f ? 1.f / sum : 0.f;
+        }
         ld_group_sync();
         if (n_t > 0) {
             tcgen05_fence_after();
-            float* o_s = reinterpret_cast<float*>(c_s);            // [NH][rank]: every page of the ring has been used
-#pragma unroll 1
-            for (int mb = 0; mb < a.m_blocks; ++mb) {
+            const int row = (a.rank + 3) / 4 * 4;
+            float* o_s = reinterpret_cast<float*>(c_s);            // [NH][row]: every page of the ring has been used
+            const int hn = a.splits > 1 ? NH : min(NH, a.heads - h0);
+            for (int mb = 0; mb < a.m_blocks; mb += 2) {           // two blocks' reads in flight
                 const int d = mb * 128 + quarter * 32 + lane;
+                const bool on0 = d < a.rank, on1 = mb + 1 < a.m_blocks && d + 128 < a.rank;
 #pragma unroll
                 for (int c0 = 0; c0 < NH; c0 += 16) {
-                    uint32_t r[16];
-                    tcgen05_ld16(tmem_o + mb * NH + lane_base + c0, r);
+                    uint32_t r[2][16];
+                    tcgen05_ld16(tmem_o + mb * NH + lane_base + c0, r[0]);
+                    if (mb + 1 < a.m_blocks) tcgen05_ld16(tmem_o + (mb + 1) * NH + lane_base + c0, r[1]);
                     tcgen05_wait_ld();
-                    if (d < a.rank) {
+                    if (a.splits > 1) {
+                        float* o = o_s + c0 * row + d;
 #pragma unroll
-                        for (int j = 0; j < 16; ++j) {
-                            const int h = c0 + j;
-                            if (a.splits == 1) {
-                                if (h0 + h < a.heads)
-                                    a.out[((size_t)t * a.heads + h0 + h) * a.rank + d] = __float2bfloat16_rn(__uint_as_float(r[j]) / l_s[h]);
-                            } else {
-                                o_s[h * a.rank + d] = __uint_as_float(r[j]);
-                            }
+                        for (int j = 0; j < 16; ++j, o += row) {
+                            if (on0) o[0] = __uint_as_float(r[0][j]);
+                            if (on1) o[128] = __uint_as_float(r[1][j]);
+                        }
+                        continue;
+                    }
+                    __nv_bfloat16* o = a.out + ((size_t)t * a.heads + h0 + c0) * a.rank + d;
+                    if (c0 + 16 <= hn) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j, o += a.rank) {
+                            if (on0) o[0] = __float2bfloat16_rn(__uint_as_float(r[0][j]) * corr_s[c0 + j]);
+                            if (on1) o[128] = __float2bfloat16_rn(__uint_as_float(r[1][j]) * corr_s[c0 + j]);
+                        }
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j, o += a.rank) {
+                            if (c0 + j < hn && on0) o[0] = __float2bfloat16_rn(__uint_as_float(r[0][j]) * corr_s[c0 + j]);
+                            if (c0 + j < hn && on1) o[128] = __float2bfloat16_rn(__uint_as_float(r[1][j]) * corr_s[c0 + j]);
                         }
                     }
                 }
@@ -317,36 +371,62 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
         }
     }
     if (a.splits > 1) {
-        // ---- the CTAs of a token merge: every one finishes a share of the (head, dimension) results
+        // ---- the CTAs of a token merge: CTA r finishes the dimensions r * per .. of all heads, from every CTA's O (in its ring's
+        // memory by now), reference and sum; 16 bytes a load, the loads of eight CTAs in flight.
         __syncthreads();
         ld_cluster_sync();
         const int tid = threadIdx.x, hn = min(NH, a.heads - h0);
-        for (int h = tid; h < hn; h += LD_THREADS) {
-            float m[LD_MAX_SPLITS], top = -INFINITY, sum = 0.f;
-            const uint32_t am = smem_u32(m_s + h), al = smem_u32(l_s + h);
-            for (int r = 0; r < a.splits; ++r) { m[r] = ld_remote(ld_peer(am, r)); top = fmaxf(top, m[r]); }
+        const int row = (a.rank + 3) / 4 * 4, per = ((a.rank + a.splits - 1) / a.splits + 3) / 4 * 4;
+        const int dn4 = (max(0, min(per, a.rank - split * per)) + 3) / 4;
+        auto pull = [&](int e, int r0, float4* x) {
+            const int h = e / dn4, d4 = e - h * dn4;
+            const uint32_t at = smem_u32(c_s) + (uint32_t)(h * row + split * per + 4 * d4) * 4;
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+                if (r0 + u < a.splits) x[u] = ld_pull4(ld_peer(at, r0 + u));
+        };
+        for (int e = tid; e < a.splits * NH; e += LD_THREADS)
+            *reinterpret_cast<float2*>(wts_s + 2 * e) = ld_pull2(ld_peer(smem_u32(l_s + 2 * (e % NH)), e / NH));
+        float4 x[8];
+        if (tid < hn * dn4) pull(tid, 0, x);                       // under way while the weights are made
+        __syncthreads();
+        if (tid < NH) {
+            float top = -INFINITY, sum = 0.f;
+#pragma unroll 4
+            for (int r = 0; r < a.splits; ++r) top = fmaxf(top, wts_s[(r * NH + tid) * 2]);
+#pragma unroll 4
             for (int r = 0; r < a.splits; ++r) {
-                m[r] = m[r] == -INFINITY ? 0.f : at_exp2(m[r] - top);
-                sum += m[r] * (m[r] > 0.f ? ld_remote(ld_peer(al, r)) : 0.f);
+                const float m = wts_s[(r * NH + tid) * 2];
+                const float w = m == -INFINITY ? 0.f : at_exp2(m - top);
+                sum = fmaf(w, wts_s[(r * NH + tid) * 2 + 1], sum);
+                wts_s[(r * NH + tid) * 2] = w;
             }
             const float inv = sum > 0.f ? 1.f / sum : 0.f;
-            for (int r = 0; r < a.splits; ++r) wts_s[r * NH + h] = m[r] * inv;
+#pragma unroll 4
+            for (int r = 0; r < a.splits; ++r) wts_s[(r * NH + tid) * 2] *= inv;
         }
         __syncthreads();
-        const int n4 = hn * a.rank / 4, share = (n4 + a.splits - 1) / a.splits;
-        const int e1 = min(n4, (split + 1) * share);
-        for (int e = split * share + tid; e < e1; e += LD_THREADS) {
-            const int h = 4 * e / a.rank, d = 4 * e - h * a.rank;
-            const uint32_t ao = smem_u32(c_s) + (uint32_t)(h * a.rank + d) * 4;
+        for (int e = tid; e < hn * dn4; e += LD_THREADS) {
+            const int h = e / dn4, d = split * per + 4 * (e - h * dn4);
             float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-            for (int r = 0; r < a.splits; ++r) {                   // ranks in order
-                const float w = wts_s[r * NH + h];
-                if (w != 0.f) {                                    // (a CTA without a page has nothing in its buffer)
-                    const float4 v = ld_remote4(ld_peer(ao, r));
-                    o.x = fmaf(w, v.x, o.x); o.y = fmaf(w, v.y, o.y); o.z = fmaf(w, v.z, o.z); o.w = fmaf(w, v.w, o.w);
+            for (int r0 = 0; r0 < a.splits; r0 += 8) {             // ranks in order
+                if (e != tid || r0 > 0) pull(e, r0, x);
+#pragma unroll
+                for (int u = 0; u < 8; ++u) {
+                    const float w = r0 + u < a.splits ? wts_s[((r0 + u) * NH + h) * 2] : 0.f;
+                    if (w != 0.f) {                                // (a CTA without a page has nothing in its memory)
+                        o.x = fmaf(w, x[u].x, o.x); o.y = fmaf(w, x[u].y, o.y); o.z = fmaf(w, x[u].z, o.z); o.w = fmaf(w, x[u].w, o.w);
+                    }
                 }
             }
-            *reinterpret_cast<uint2*>(a.out + ((size_t)t * a.heads + h0 + h) * a.rank + d) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+            __nv_bfloat16* dst = a.out + ((size_t)t * a.heads + h0 + h) * a.rank + d;
+            if (a.rank % 4 == 0) {
+                *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+            } else {
+                const float v[4] = {o.x, o.y, o.z, o.w};
+                for (int i = 0; i < 4; ++i)
+                    if (d + i < a.rank) dst[i] = __float2bfloat16_rn(v[i]);
+            }
         }
         ld_cluster_sync();                                         // nobody leaves while its memory is read
     }
@@ -363,19 +443,19 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
 struct LatentDecodePlan { int nh, nb, m_blocks, stages, cols; size_t smem; };
 
 static bool ld_plan(int heads, int rank, int ld, LatentDecodePlan* p) {
-    if (heads < 1 || rank < 4 || rank % 4 || ld < rank || ld % 8) return false;
+    if (heads < 1 || rank < 1 || ld < rank || ld % 8) return false;
     const int nb = (ld + 63) / 64, mb = (rank + 127) / 128;
     for (int nh = heads <= 16 ? 16 : (heads <= 32 ? 32 : 64); nh >= 16; nh /= 2) {
         int cols = 32;
         while (cols < (2 + mb) * nh) cols *= 2;
         if (cols > 512) continue;
-        const size_t fixed = (size_t)nb * nh * 128 + 2 * nh * 128 + (size_t)(7 + LD_MAX_SPLITS) * nh * 4 + 15 * 8 + 16;
+        const size_t fixed = (size_t)nb * nh * 128 + 2 * nh * 128 + (size_t)(8 + 2 * LD_MAX_SPLITS) * nh * 4 + 15 * 8 + 16;
         const size_t tile = (size_t)nb * LD_PAGE_BLOCK, limit = 227 * 1024;
         if (fixed + tile > limit) continue;
         int stages = (int)((limit - fixed) / tile);
         if (stages > 4) stages = 4;
-        // the merge keeps [nh][rank] floats where the ring was
-        if ((size_t)nh * rank * 4 > stages * tile) continue;
+        // the merge keeps [nh][rank in whole fours] floats where the ring was
+        if ((size_t)nh * (rank + 4) * 4 > stages * tile) continue;
         *p = LatentDecodePlan{nh, nb, mb, stages, cols, fixed + stages * tile};
         // as many CTAs on a multiprocessor as its tensor memory serves, no more: a CTA that waits for tensor memory while its
         // cluster's other CTAs hold theirs could wait for good

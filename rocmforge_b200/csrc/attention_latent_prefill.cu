@@ -24,7 +24,7 @@ struct LatentPrefill {
     const int *seq_start, *seq_nnew, *cu_q, *cu_k;
     int dim, rot, vdim, rank, v_col;
     int nq, nr, nv;                                  // 64-column blocks of a head's unrotated part, rotated part, values
-    int v_stages;
+    int k_stages, v_stages;
     int tmem_cols;
     float scale;
     int span;
@@ -43,8 +43,8 @@ attention_latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const
     extern __shared__ __align__(1024) uint8_t smem[];                  // no static shared memory: the window starts aligned
     const int nb = a.nq + a.nr;
     uint8_t* q_s = smem;                                               // [nb][128][128 B]
-    uint8_t* k_s = q_s + (size_t)nb * QB;                              // [2][nb][64][128 B]
-    uint8_t* v_s = k_s + (size_t)2 * nb * KB;                          // [v_stages][nv][64][128 B]
+    uint8_t* k_s = q_s + (size_t)nb * QB;                              // [k_stages][nb][64][128 B]
+    uint8_t* v_s = k_s + (size_t)a.k_stages * nb * KB;                 // [v_stages][nv][64][128 B]
     uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + (size_t)a.v_stages * a.nv * KB);
     // q_full, k_full[2], k_free[2], s_full[2], p_ready[2], pv_done[2], v_full[2], v_free[2]; p_ready and pv_done alternate
     // from tile to tile so that no barrier completes two phases between two looks of one of its waiters
@@ -99,15 +99,16 @@ attention_latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const
             for (int b = 0; b < a.nq; ++b) tma_load_2d(smem_u32(q_s + b * QB), &map_q, qc + b * 64, row_base, b_q);
             for (int b = 0; b < a.nr; ++b) tma_load_2d(smem_u32(q_s + (a.nq + b) * QB), &map_q, qc + a.dim + b * 64, row_base, b_q);
             for (int t = 0; t < n_kt; ++t) {
-                const int st = t & 1, row = key_base + (kt_lo + t) * LP_BN;
-                uint8_t* kd = k_s + (size_t)st * nb * KB;
-                if (!mbar_wait(b_kfree + 8 * st, ((t >> 1) & 1) ^ 1, &abort_flag)) break;
-                mbar_expect_tx(b_kfull + 8 * st, nb * KB);
+                const int row = key_base + (kt_lo + t) * LP_BN;
+                const int sk = a.k_stages == 2 ? t & 1 : 0, use_k = a.k_stages == 2 ? t >> 1 : t;
+                uint8_t* kd = k_s + (size_t)sk * nb * KB;
+                if (!mbar_wait(b_kfree + 8 * sk, (use_k & 1) ^ 1, &abort_flag)) break;
+                mbar_expect_tx(b_kfull + 8 * sk, nb * KB);
                 for (int b = 0; b < a.nq; ++b)
-                    tma_load_2d(smem_u32(kd + b * KB), &map_kv, head * a.dim + b * 64, row, b_kfull + 8 * st);
+                    tma_load_2d(smem_u32(kd + b * KB), &map_kv, head * a.dim + b * 64, row, b_kfull + 8 * sk);
                 for (int b = 0; b < a.nr; ++b)
-                    tma_load_2d(smem_u32(kd + (a.nq + b) * KB), &map_lat, a.rank + b * 64, row, b_kfull + 8 * st);
-                const int sv = a.v_stages == 2 ? st : 0, use = a.v_stages == 2 ? t >> 1 : t;
+                    tma_load_2d(smem_u32(kd + (a.nq + b) * KB), &map_lat, a.rank + b * 64, row, b_kfull + 8 * sk);
+                const int sv = a.v_stages == 2 ? t & 1 : 0, use = a.v_stages == 2 ? t >> 1 : t;
                 uint8_t* vd = v_s + (size_t)sv * a.nv * KB;
                 if (!mbar_wait(b_vfree + 8 * sv, (use & 1) ^ 1, &abort_flag)) break;
                 mbar_expect_tx(b_vfull + 8 * sv, a.nv * KB);
@@ -117,22 +118,24 @@ attention_latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const
         }
     } else if (warp == 1) {
         // ---------------- MMA issuer
-        if (lane == 0) {
+        if (elect_one()) {
             const uint32_t idesc_s = lp_idesc(LP_BN, 0), idesc_o = lp_idesc(a.vdim, 1);
-            const int ks_dim = a.dim >> 4, ks_rot = (a.rot + 15) >> 4;
+            const int ks_dim = a.dim >> 4, ks_all = ks_dim + ((a.rot + 15) >> 4);
             auto issue_s = [&](int t) -> bool {          // the scores of tile t + 1 are computed under the softmax of tile t
-                const int st = t & 1;
-                if (!mbar_wait(b_kfull + 8 * st, (t >> 1) & 1, &abort_flag)) return false;
+                const int st = t & 1, sk = a.k_stages == 2 ? st : 0, use_k = a.k_stages == 2 ? t >> 1 : t;
+                if (!mbar_wait(b_kfull + 8 * sk, use_k & 1, &abort_flag)) return false;
                 tcgen05_fence_after();
-                const uint32_t k_t = smem_u32(k_s + (size_t)st * nb * KB), q_t = smem_u32(q_s), d = tmem_s + st * LP_BN;
-                for (int ks = 0; ks < ks_dim; ++ks)
-                    tcgen05_mma_bf16(d, make_smem_desc(q_t + (ks >> 2) * QB + (ks & 3) * 32),
-                                     make_smem_desc(k_t + (ks >> 2) * KB + (ks & 3) * 32), idesc_s, ks ? 1u : 0u);
-                for (int ks = 0; ks < ks_rot; ++ks)
-                    tcgen05_mma_bf16(d, make_smem_desc(q_t + (a.nq + (ks >> 2)) * QB + (ks & 3) * 32),
-                                     make_smem_desc(k_t + (a.nq + (ks >> 2)) * KB + (ks & 3) * 32), idesc_s, (ks_dim | ks) ? 1u : 0u);
+                uint64_t kd = make_smem_desc(smem_u32(k_s + (size_t)sk * nb * KB)), qd = make_smem_desc(smem_u32(q_s));
+                const uint32_t d = tmem_s + st * LP_BN;
+                // block after block: the unrotated columns' steps, then the rotated ones' (a step is 32 bytes, 2 descriptor units)
+                for (int b = 0; b < nb; ++b, qd += QB >> 4, kd += KB >> 4) {
+                    const int left = b < a.nq ? ks_dim - 4 * b : ks_all - ks_dim - 4 * (b - a.nq);
+#pragma unroll
+                    for (int k = 0; k < 4; ++k)
+                        if (k < left) tcgen05_mma_bf16(d, qd + 2 * k, kd + 2 * k, idesc_s, (b | k) ? 1u : 0u);
+                }
                 tcgen05_commit(b_sfull + 8 * st);
-                tcgen05_commit(b_kfree + 8 * st);
+                tcgen05_commit(b_kfree + 8 * sk);
                 return true;
             };
             bool ok = mbar_wait(b_q, 0, &abort_flag);
@@ -285,15 +288,15 @@ attention_latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const
 }
 
 // ---------------------------------------------------------------- host side
-static size_t lp_smem(int nb, int nv, int v_stages) {
-    return (size_t)nb * LP_BM * 128 + (size_t)2 * nb * LP_BN * 128 + (size_t)v_stages * nv * LP_BN * 128 + 15 * 8 + 16;
+static size_t lp_smem(int nb, int nv, int k_stages, int v_stages) {
+    return (size_t)nb * LP_BM * 128 + (size_t)k_stages * nb * LP_BN * 128 + (size_t)v_stages * nv * LP_BN * 128 + 15 * 8 + 16;
 }
 
 extern "C" {
 
 int rf_attention_latent_prefill_supported(int heads, int dim, int rot, int vdim, int rank) {
     if (heads < 1 || heads > 65535 || dim < 16 || dim % 16 || rot < 0 || rot % 8 || vdim < 16 || vdim % 16 || vdim > 256 || rank % 8) return 0;
-    if (lp_smem((dim + 63) / 64 + (rot + 63) / 64, (vdim + 63) / 64, 1) > 227 * 1024) return 0;
+    if (lp_smem((dim + 63) / 64 + (rot + 63) / 64, (vdim + 63) / 64, 1, 1) > 227 * 1024) return 0;
     return encode_fn() != nullptr;
 }
 
@@ -323,11 +326,16 @@ int rf_attention_latent_prefill(const void* q, int q_stride, int T, const void* 
     a.nq = (dim + 63) / 64; a.nr = (rot + 63) / 64; a.nv = (vdim + 63) / 64;
     a.tmem_cols = vdim <= 128 ? 256 : 512;
     a.scale = scale; a.span = span; a.status = status;
-    // two value stages where two CTAs still share a multiprocessor (or where one CTA fills it anyway), else one
+    // Stages: as many as leave room for two CTAs on a multiprocessor (half of 228 KB less the 1 KB the system keeps for each),
+    // or, where one CTA is all that fits, as many as fit.  Values come first: a tile's keys are used up a whole tile before its
+    // values are, so one stage of keys is refilled in time and one of values is not.
     const int nb = a.nq + a.nr;
-    const size_t two_ctas = 113 * 1024 + 512;        // per CTA: half of 228 KB less the 1 KB the system keeps for each
-    a.v_stages = lp_smem(nb, a.nv, 2) <= two_ctas ? 2 : (lp_smem(nb, a.nv, 1) <= two_ctas ? 1 : (lp_smem(nb, a.nv, 2) <= 227 * 1024 ? 2 : 1));
-    const size_t smem = lp_smem(nb, a.nv, a.v_stages);
+    const int forms[4][2] = {{2, 2}, {1, 2}, {2, 1}, {1, 1}};
+    a.k_stages = 0;
+    for (size_t limit : {(size_t)(113 * 1024), (size_t)(227 * 1024)})
+        for (int f = 0; f < 4 && a.k_stages == 0; ++f)
+            if (lp_smem(nb, a.nv, forms[f][0], forms[f][1]) <= limit) { a.k_stages = forms[f][0]; a.v_stages = forms[f][1]; }
+    const size_t smem = lp_smem(nb, a.nv, a.k_stages, a.v_stages);
     static size_t configured = 0;
     if (smem > configured) {
         cudaError_t ce = cudaFuncSetAttribute(attention_latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);

@@ -244,8 +244,8 @@ static int st_dispatch(const StreamsArgs& a, int rows, cudaStream_t st) {
 // products in 64-bit; a sequence's first token takes row `buckets`.  state [slots][2]: the token at position p lies at
 // p & 1, so a step of one token that runs again (launched ahead of the host and dropped) finds its previous token still
 // there.  The block of a sequence's first new token reads the state and then writes it.
-template <typename T>
-__global__ void __launch_bounds__(256)
+template <typename T, int V4>
+__global__ void __launch_bounds__(512)
 pair_embed_kernel(const T* __restrict__ table, const T* __restrict__ pairs, const int* __restrict__ ids,
                   const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ seq_slot,
                   const int* __restrict__ cu_q, int* __restrict__ state, const void* __restrict__ w, int w_is_f32,
@@ -277,15 +277,30 @@ pair_embed_kernel(const T* __restrict__ table, const T* __restrict__ pairs, cons
     const T* e = table + (size_t)id * H;
     const T* p = pairs != nullptr ? pairs + (size_t)row_s * H : nullptr;
     float ss = 0.f;
-    for (int c = threadIdx.x; c < H; c += blockDim.x) {
-        float v = Cvt<T>::to_f32(e[c]) * scale;
-        if (p != nullptr) v += Cvt<T>::to_f32(p[c]);
-        sm[c] = v;
-        ss = fmaf(v, v, ss);
+    for (int c = V4 * threadIdx.x; c < H; c += V4 * blockDim.x) {
+        float v[V4], x[V4];
+        StVec<V4>::weight(e, sizeof(T) == 4, c, v);
+        if (p != nullptr) StVec<V4>::weight(p, sizeof(T) == 4, c, x);
+#pragma unroll
+        for (int i = 0; i < V4; ++i) {
+            v[i] *= scale;
+            if (p != nullptr) v[i] += x[i];
+            ss = fmaf(v[i], v[i], ss);
+        }
+        StVec<V4>::store(sm + c, v);
     }
     const float r = w != nullptr ? rsqrtf(block_sum(ss, red) / (float)H + eps) : 1.f;
     float* o = out + (size_t)t * H;
-    for (int c = threadIdx.x; c < H; c += blockDim.x) o[c] = w != nullptr ? sm[c] * r * load_vec(w, w_is_f32, c) : sm[c];
+    for (int c = V4 * threadIdx.x; c < H; c += V4 * blockDim.x) {      // a thread reads what it wrote
+        float v[V4], x[V4];
+        StVec<V4>::load(sm + c, v);
+        if (w != nullptr) {
+            StVec<V4>::weight(w, w_is_f32, c, x);
+#pragma unroll
+            for (int i = 0; i < V4; ++i) v[i] *= r * x[i];
+        }
+        StVec<V4>::store(o + c, v);
+    }
 }
 
 template <typename T>
@@ -299,13 +314,18 @@ static int launch_pair_embed(const void* table, const void* pairs, const int* id
         return RF_ERR_BAD_ARG;
     const size_t smem = (size_t)(H + 34) * sizeof(float);
     if (smem > 200 * 1024) return RF_ERR_UNSUPPORTED;
-    static size_t configured = 48 * 1024;
-    if (smem > configured) {
-        cudaError_t e = cudaFuncSetAttribute(pair_embed_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    auto whole = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+    const bool vec = H % 4 == 0 && whole(table) && whole(pairs) && whole(w) && whole(out);
+    auto kernel = vec ? pair_embed_kernel<T, 4> : pair_embed_kernel<T, 1>;
+    static size_t configured[2] = {48 * 1024, 48 * 1024};
+    if (smem > configured[vec]) {
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
-        configured = smem;
+        configured[vec] = smem;
     }
-    rf_launch(pair_embed_kernel<T>, dim3(T_), dim3(256), smem, st, reinterpret_cast<const T*>(table), reinterpret_cast<const T*>(pairs),
+    int threads = ((vec ? H / 4 : H) + 31) / 32 * 32;
+    threads = threads < 64 ? 64 : (threads > 512 ? 512 : threads);
+    rf_launch(kernel, dim3(T_), dim3(threads), smem, st, reinterpret_cast<const T*>(table), reinterpret_cast<const T*>(pairs),
               ids, tok_seq, tok_pos, seq_slot, cu_q, state, w, w_is_f32, out, H, V, scale, mul_prev, mul_cur, buckets, eps);
     RF_LAUNCH_CHECK();
     return 0;

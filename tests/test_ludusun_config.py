@@ -128,7 +128,7 @@ def test_keys_that_serve_as_values_are_stored_once():
     assert shared.k_pages.data_ptr() == shared.v_pages.data_ptr() and plain.k_pages.data_ptr() != plain.v_pages.data_ptr()
     assert sum(g.storage.numel() for g in cache.groups) == 3 * plain.k_pages.numel()
     with pytest.raises(ValueError):
-        KVRequest(2, 16, v_head_dim=8, values_are_keys=True)
+        KVRequest(2, 16, v_head_dim=24, values_are_keys=True)
 
 
 def test_the_norm_adds_its_offset_once_in_32_bits():
