@@ -446,3 +446,82 @@ def write_ludusun(cfg: dict, folder: str, dtype: str = "float32") -> None:
     c, raw = ludusun_config(cfg)
     dt = {"float32": torch.float32, "bfloat16": torch.bfloat16}[dtype]
     rf.write_model_folder(folder, raw, architecture_for("Ludusun").build(c).param_specs(), cfg["seed"], dt)
+
+
+# --------------------------------------------------------------------------- Gedilorn
+
+def _latent_cache(kind, *, heads, dim, rot_dim, vdim, kv_rank, scale, base=None, scaling=None, mlp, weights_of=None):
+    mix = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "scale": scale}
+    if rot_dim:
+        mix["rot"] = {"dims": rot_dim, "base": base}
+        if scaling is not None:
+            mix["rot"]["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    L = {"type": "latent_attention_2" if kind == "gated" else "latent_attention", "mixer": mix, "mlp": mlp}
+    if weights_of is not None:
+        L["weights_of"] = weights_of
+    return L
+
+
+def _again(L, j):
+    """The same layer once more with layer j's weights."""
+    return dict(L, weights_of=j)
+
+
+# Sizes that differ from each other in every respect: both kinds of layer first; one head, a few, more than 16, 32 and 64
+# (the latent decode kernel's groups); head parts that no tensor-core kernel takes (odd latents, parts of 10 and 6) and parts
+# it takes with every remainder (unrotated 16 to 128, rotated 0, 8, 16, 24 and 64, values from 14 to 144, latents from 21 to
+# 512); frequencies stretched and not; layers without feed-forward; weights used by one later layer, by several, and by an
+# earlier one; 1, 2, 3, 5 and 9 streams and the ordinary residual; with and without a table of pairs, tables of few buckets
+# and of more than the vocabulary, multipliers larger than the buckets; logits scaled and not; a width that no tensor-core
+# product takes.
+_GA = [_latent_cache("gated", heads=3, dim=10, rot_dim=6, vdim=14, kv_rank=21, scale=0.3, base=50.0, scaling=(3.0, 24, 4.0, 1.0), mlp=_dense(40)),
+       _latent_cache("plain", heads=1, dim=16, rot_dim=0, vdim=8, kv_rank=12, scale=0.25, mlp=None)]
+GEDILORN_A = dict(seed=51, architecture="Gedilorn", vocab=96, width=64, norm={"eps": 1e-5}, streams=2, logit_scale=0.7,
+                  embedding={"scale": 3.0, "bigram": {"buckets": 37, "mul_prev": 1009, "mul_cur": 53}},
+                  layers=[_GA[0], _GA[1], _again(_GA[0], 0), _again(_GA[0], 0)])
+_GB = [_latent_cache("plain", heads=4, dim=32, rot_dim=16, vdim=32, kv_rank=64, scale=0.2, base=1e4, mlp=_dense(96)),
+       _latent_cache("gated", heads=2, dim=64, rot_dim=8, vdim=48, kv_rank=40, scale=0.12, base=1e6, scaling=(8.0, 512, 32.0, 1.0), mlp=_dense(64))]
+GEDILORN_B = dict(seed=52, architecture="Gedilorn", vocab=200, width=128, norm={"eps": 1e-6}, embedding={"scale": 1.0},
+                  layers=[_GB[0], _GB[1], _again(_GB[1], 1)])
+_GC = [_latent_cache("plain", heads=5, dim=48, rot_dim=24, vdim=96, kv_rank=136, scale=0.13, base=1e4, scaling=(2.0, 128, 16.0, 2.0), mlp=_dense(320)),
+       _latent_cache("gated", heads=20, dim=16, rot_dim=8, vdim=16, kv_rank=72, scale=0.2, base=500.0, mlp=_dense(128)),
+       _latent_cache("gated", heads=2, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=0.07, base=1e6, scaling=(4.0, 256, 32.0, 1.0), mlp=None)]
+GEDILORN_C = dict(seed=53, architecture="Gedilorn", vocab=304, width=256, norm={"eps": 1e-6}, streams=3, logit_scale=2.0,
+                  embedding={"scale": 12.0, "bigram": {"buckets": 600, "mul_prev": 31, "mul_cur": 17}},
+                  layers=[_again(_GC[0], 2), _GC[1], _GC[0], _GC[2], _again(_GC[1], 1), _again(_GC[2], 3)])
+_GD = [_latent_cache("gated", heads=40, dim=16, rot_dim=16, vdim=144, kv_rank=200, scale=0.2, base=1e4, mlp=_dense(24)),
+       _latent_cache("plain", heads=7, dim=80, rot_dim=0, vdim=16, kv_rank=64, scale=0.1, mlp=_dense(16))]
+GEDILORN_D = dict(seed=54, architecture="Gedilorn", vocab=130, width=100, norm={"eps": 3e-6}, streams=9,
+                  embedding={"bigram": {"buckets": 1, "mul_prev": 5, "mul_cur": 3}}, layers=[_GD[1], _GD[0]])
+_GE = [_latent_cache("plain", heads=70, dim=16, rot_dim=8, vdim=16, kv_rank=56, scale=0.25, base=1e3, mlp=_dense(64)),
+       _latent_cache("gated", heads=8, dim=64, rot_dim=40, vdim=112, kv_rank=320, scale=0.1, base=1e5, scaling=(16.0, 64, 8.0, 0.5), mlp=_dense(136))]
+GEDILORN_E = dict(seed=55, architecture="Gedilorn", vocab=150, width=192, norm={"eps": 1e-5}, streams=5, logit_scale=0.25,
+                  embedding={"scale": 0.5, "bigram": {"buckets": 211, "mul_prev": 2, "mul_cur": 1}}, layers=[_GE[0], _GE[1]])
+GEDILORN_F = dict(seed=56, architecture="Gedilorn", vocab=120, width=64, norm={"eps": 1e-6}, streams=1,
+                  embedding={"scale": 2.0, "bigram": {"buckets": 90, "mul_prev": 7, "mul_cur": 11}}, layers=[_GB[0], _again(_GB[0], 0)])
+GEDILORN_CONFIGS = {"GA": GEDILORN_A, "GB": GEDILORN_B, "GC": GEDILORN_C, "GD": GEDILORN_D, "GE": GEDILORN_E, "GF": GEDILORN_F}
+
+
+def gedilorn_config(cfg: dict):
+    """(typed configuration, the dict that goes into config.json)."""
+    from rocmforge_b200.config import architecture_for
+    raw = {k: v for k, v in cfg.items() if k != "seed"}
+    return architecture_for("Gedilorn").config_cls.from_dict(raw), raw
+
+
+def write_gedilorn(cfg: dict, folder: str, dtype: str = "float32") -> None:
+    """Matrices with a standard deviation of 1.2 / sqrt(inputs), so that scores spread, keys differ and gates are not all a half;
+    norm weights around one, not one; every stream's coefficients of its own."""
+    import dataclasses
+    import rocmforge_b200 as rf
+    from rocmforge_b200.config import architecture_for
+    c, raw = gedilorn_config(cfg)
+    specs = {}
+    for name, s in architecture_for("Gedilorn").build(c).param_specs().items():
+        if s.kind == "matrix":
+            s = dataclasses.replace(s, std=0.5 if name in ("embed", "bigram") else 1.2 / s.shape[1] ** 0.5)
+        elif s.init == "ones":
+            s = dataclasses.replace(s, init="normal", mean=1.0, std=0.2)
+        specs[name] = s
+    dt = {"float32": torch.float32, "bfloat16": torch.bfloat16}[dtype]
+    rf.write_model_folder(folder, raw, specs, cfg["seed"], dt)
