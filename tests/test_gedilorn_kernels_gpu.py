@@ -120,3 +120,318 @@ def test_relu_gated_product(M, N, K):
         tol = 1e-4 if y.dtype == F32 else 1e-2
         assert y.shape == want.shape and (y.double() - want).abs().max() < tol * want.abs().max()
     status_clean()
+
+
+# --------------------------------------------------------------------------- latents on their way into the cache
+
+def _positions(lens, starts, extra=3, seed=0):
+    """(tok_seq, tok_pos, seq_slot, block_table, n_pages) of sequences that bring lens[i] tokens from starts[i] on; pages shuffled."""
+    g = torch.Generator().manual_seed(seed)
+    B = len(lens)
+    need = [(s + n + 63) // 64 for s, n in zip(starts, lens)]
+    n_pages = sum(need) + extra
+    order = torch.randperm(n_pages, generator=g).tolist()
+    bt = torch.full((B + 2, max(need)), -1, dtype=torch.int32)
+    slots = [(2 * i + 1) % (B + 2) for i in range(B)] if (B + 2) % 2 else list(range(1, B + 1))
+    at = 0
+    for i in range(B):
+        bt[slots[i], :need[i]] = torch.tensor(order[at:at + need[i]], dtype=torch.int32)
+        at += need[i]
+    seq = [i for i, n in enumerate(lens) for _ in range(n)]
+    pos = [s + k for s, n in zip(starts, lens) for k in range(n)]
+    return ints(seq), ints(pos), ints(slots), bt.to(DEV), n_pages
+
+
+@pytest.mark.parametrize("H,D,R,K", [(3, 10, 6, 21), (1, 16, 0, 12), (5, 48, 24, 136), (20, 128, 64, 512), (2, 8, 2, 3)])
+@pytest.mark.parametrize("dt", [F32, BF16])
+def test_the_cache_row_and_the_query_parts(H, D, R, K, dt):
+    """Norm of the latent's part only, rotation of neighbouring pairs with stretched frequencies and a magnitude, zeros behind; rows
+    at the right places of shuffled pages and nothing else touched; from the product's matrix and from partial sums; queries left
+    in place (turned where they lie) and taken out; the gate's columns."""
+    from rocmforge_b200 import kernels
+    from rocmforge_b200.parts import POSITIONS
+    torch.manual_seed(H)
+    lens, starts = [5, 1, 70], [0, 63, 3]
+    seq, pos, slots, bt, n_pages = _positions(lens, starts)
+    T, G = sum(lens), 24
+    q_n, ld = H * (D + R), (K + R + 7) // 8 * 8
+    down_col = (q_n + 7) // 8 * 8
+    gate_col = (down_col + K + R + 7) // 8 * 8
+    src = torch.randn(T, gate_col + G, device=DEV).to(dt)
+    w = (torch.rand(K, device=DEV) + 0.5).to(dt)
+    rot = None
+    if R:
+        enc = POSITIONS.build("rope_yarn", head_dim=R, theta=100.0, interleaved=True, factor=4.0, original=64, fast=8.0, slow=1.0)
+        enc.prepare(DEV)
+        rot = enc.rotation()
+    x = src.double().cpu()
+    c = P.rms_norm(x[:, down_col:down_col + K], w.double().cpu(), 1e-5)
+    heads = x[:, :q_n].reshape(T, H, D + R)
+    kr, qr = x[:, down_col + K:down_col + K + R], heads[..., D:]
+    if R:
+        f, mag = P.stretched_frequencies(R, 100.0, dict(factor=4.0, original=64, fast=8.0, slow=1.0))
+        kr, qr = P.turn_neighbours(kr, pos.cpu(), f, mag), P.turn_neighbours(qr, pos.cpu(), f, mag)
+    want = torch.cat([c, kr, torch.zeros(T, ld - K - R, dtype=torch.float64)], dim=1)
+    tol = 2e-5 if dt == F32 else 1e-2
+
+    def near(got, ref):
+        assert got.numel() == 0 or (got.double().cpu() - ref).abs().max() <= tol * max(1.0, float(ref.abs().max()))
+    for form in ("matrix", "parts", "in place"):
+        pages = torch.full((n_pages, 1, 64, ld), 7.0, device=DEV, dtype=dt)
+        a = src.clone()
+        if form == "parts":
+            half = torch.randn_like(a.float())
+            a = torch.stack([a.float() - half, half])
+        rows = torch.full((T, ld), 3.0, device=DEV, dtype=dt)
+        q_dim = torch.zeros(T, H, D, device=DEV, dtype=dt)
+        folded = torch.full((T, H, ld), 5.0, device=DEV, dtype=dt)
+        q_rot = folded[:, :, K:] if form != "in place" else a[:, :q_n].unflatten(1, (H, D + R))[:, :, D:]
+        gate = torch.zeros(T, G, device=DEV, dtype=dt)
+        kernels.latent_write(a, q_col=0, down_col=down_col, heads=H, dim=D, rot=R, rank=K, norm_weight=w, eps=1e-5, rotation=rot,
+                             tok_seq=seq, tok_pos=pos, seq_slot=slots, block_table=bt, pages=pages, compute_dtype=dt, rows=rows,
+                             q_dim=q_dim if form != "in place" else None,
+                             q_rot=q_rot if q_rot.shape[2] else None, gate_col=gate_col, gate=gate)
+        near(rows, want)
+        flat = pages.view(n_pages * 64, ld)
+        at = bt[slots.long()[seq.long()], (pos // 64).long()].long() * 64 + (pos % 64).long()
+        assert torch.equal(flat[at], rows)
+        untouched = torch.ones(n_pages * 64, dtype=torch.bool, device=DEV)
+        untouched[at] = False
+        assert (flat[untouched] == 7.0).all()
+        near(gate, x[:, gate_col:gate_col + G])
+        near(q_rot[:, :, :R], qr)
+        if form == "in place":
+            assert torch.equal(a[:, :q_n].unflatten(1, (H, D + R))[:, :, :D], src[:, :q_n].unflatten(1, (H, D + R))[:, :, :D])
+        else:
+            near(q_dim, heads[..., :D])
+            assert (folded[:, :, :K] == 5.0).all() and (folded[:, :, K + R:] == 0).all()
+
+
+def test_rows_of_whole_sequences_are_gathered_in_order():
+    from rocmforge_b200 import kernels
+    lens = [1, 64, 65, 200]
+    seq, pos, slots, bt, n_pages = _positions(lens, [0] * 4)
+    pages = torch.randn(n_pages, 1, 64, 24, device=DEV).to(BF16)
+    cu = ints([0] + torch.tensor(lens).cumsum(0).tolist())
+    got = kernels.latent_gather(pages, cu, slots, bt, sum(lens))
+    at = bt[slots.long()[seq.long()], (pos // 64).long()].long() * 64 + (pos % 64).long()
+    assert torch.equal(got, pages.view(-1, 24)[at])
+
+
+@pytest.mark.parametrize("T", [1, 5, 16, 17, 70, 130])
+@pytest.mark.parametrize("H,N,K", [(1, 8, 12), (3, 21, 10), (5, 136, 48), (16, 512, 128), (16, 128, 512), (2, 100, 72)])
+def test_a_matrix_per_head(T, H, N, K):
+    """Strided inputs and outputs (other columns untouched), with and without the gate, sizes that are no multiple of a tile."""
+    from rocmforge_b200 import kernels
+    torch.manual_seed(T)
+    for dt in (F32, BF16):
+        pad = 8 - K % 8 if K % 8 else 8
+        x = torch.randn(T, H, K + pad, device=DEV).to(dt)[:, :, :K]
+        w = (torch.randn(H, N, K, device=DEV) / K ** 0.5).to(dt)
+        out = torch.full((T, H, N + 3), 9.0, device=DEV, dtype=dt)
+        gate = torch.randn(T, H * N + 8, device=DEV).to(dt)[:, :H * N]
+        want = torch.einsum("thk,hnk->thn", x.double(), w.double())
+        tol = 1e-5 if dt == F32 else 1e-2
+        kernels.head_product(x, w, out=out)
+        assert (out[:, :, :N].double() - want).abs().max() < tol * want.abs().max() and (out[:, :, N:] == 9.0).all()
+        got = kernels.head_product(x, w, gate=gate)
+        want = want * torch.sigmoid(gate.double()).view(T, H, N)
+        assert (got.double() - want).abs().max() < tol * want.abs().max()
+
+
+# --------------------------------------------------------------------------- attention
+
+def _softmax_rows(q, keys, vals, scale, upto):
+    """q [n, H, L], keys [T, H or 1, L], vals [T, H or 1, V]: row r sees keys 0 .. upto[r]; float64."""
+    n, H, _ = q.shape
+    out = []
+    for h in range(H):
+        k, v = keys[:, h % keys.shape[1]], vals[:, h % vals.shape[1]]
+        s = (q[:, h] @ k.T) * scale
+        hidden = torch.arange(k.shape[0], device=s.device)[None, :] > torch.as_tensor(upto, device=s.device)[:, None]
+        out.append(torch.softmax(s.masked_fill(hidden, float("-inf")), dim=-1) @ v)
+    return torch.stack(out, dim=1)
+
+
+DECODE_SIZES = [(1, 64, 16), (3, 21, 6), (16, 512, 64), (17, 136, 24), (32, 200, 0), (40, 64, 8), (70, 56, 8), (128, 128, 64), (6, 192, 0),
+                (2, 1024, 64)]
+
+
+@pytest.mark.parametrize("H,K,R", DECODE_SIZES)
+def test_single_tokens_over_cached_latents(H, K, R):
+    """Sequences of 1 to 700 positions in shuffled pages whose other rows are NaN (pages not owned, positions not written), every
+    number of CTAs a token, against the softmax written out in float64; the generic kernel on the same rows in 32-bit."""
+    from rocmforge_b200 import kernels
+    torch.manual_seed(H + K)
+    ends = [1, 2, 16, 17, 63, 64, 65, 128, 130, 321, 700]
+    ld = (K + R + 7) // 8 * 8
+    B = len(ends)
+    seq, pos, slots, bt, n_pages = _positions(ends, [0] * B)
+    at = bt[slots.long()[seq.long()], (pos // 64).long()].long() * 64 + (pos % 64).long()
+    for dt in (F32, BF16):
+        pages = torch.full((n_pages, 1, 64, ld), float("nan"), device=DEV, dtype=dt)
+        rows = torch.randn(sum(ends), ld, device=DEV).to(dt)
+        rows[:, K + R:] = 0
+        pages.view(-1, ld)[at] = rows
+        q = (torch.randn(B, H, ld, device=DEV) * 0.6).to(dt)
+        scale = 2.0 / (K + R) ** 0.5
+        tok_seq, tok_pos, start = ints(range(B)), ints(e - 1 for e in ends), ints(max(e - 1, 0) for e in ends)
+        want, a = [], 0
+        for i, e in enumerate(ends):
+            k = rows[a:a + e].double()[:, None]
+            want.append(_softmax_rows(q[i:i + 1].double(), k, k[..., :K], scale, [e - 1])[0])
+            a += e
+        want = torch.stack(want)
+        got = kernels.attention_generic(q.view(B, H * ld), H, 1, ld, pages, pages[..., :K], tok_seq, tok_pos, slots, bt, scale, None,
+                                        v_head_dim=K).view(B, H, K).double()
+        assert (got - want).abs().max() < (1e-5 if dt == F32 else 2e-2) * want.abs().max(), "generic"
+        if dt == F32:
+            continue
+        assert kernels.attention_latent_decode_groups(H, K, ld) == -(-H // (16 if H <= 16 else 32 if H <= 32 else 64)) or K > 512
+        for splits in (1, 2, 3, 4, 8, None):
+            got = kernels.attention_latent_decode(q, pages, tok_seq, tok_pos, slots, start, bt, rank=K, scale=scale, splits=splits,
+                                                  longest=max(ends)).double()
+            err = (got - want).abs().amax(dim=(1, 2))
+            assert err.max() < 2e-2 * want.abs().max(), f"{splits} CTAs a token: context of {ends[int(err.argmax())]}"
+    status_clean()
+
+
+@pytest.mark.parametrize("splits", [1, 2, 8])
+@pytest.mark.parametrize("i,j", [(699, 0), (699, 63), (699, 64), (699, 639), (699, 640), (130, 1), (255, 128), (256, 127), (64, 0), (63, 63)])
+def test_a_far_latent_among_hundreds(i, j, splits):
+    """One position's row stands out and is found, with its own values; the row just behind the query would stand out more."""
+    from rocmforge_b200 import kernels
+    torch.manual_seed(i * 1000 + j)
+    T, H, K, R = 702, 5, 96, 16
+    rows = torch.randn(T, K + R, device=DEV) * 0.05
+    rows[:, 0] = 0
+    rows[j, 0], rows[i + 1, 0] = 4.0, 8.0
+    rows[j, 1:K] = torch.randn(K - 1, device=DEV)
+    rows[i + 1, 1:K] = 1000.0
+    q = torch.zeros(1, H, K + R, device=DEV)
+    q[..., 0] = 8.0
+    rows, q = rows.to(BF16), q.to(BF16)
+    seq, pos, slots, bt, n_pages = _positions([T], [0])
+    pages = torch.full((n_pages, 1, 64, K + R), float("nan"), device=DEV, dtype=BF16)
+    at = bt[slots.long()[seq.long()], (pos // 64).long()].long() * 64 + (pos % 64).long()
+    pages.view(-1, K + R)[at] = rows
+    got = kernels.attention_latent_decode(q, pages, ints([0]), ints([i]), slots, ints([i]), bt, rank=K, scale=1.0, splits=splits)
+    assert (got[0].float() - rows[j, :K].float()).abs().max() < 2e-2 * float(rows[j, :K].float().abs().max())
+    status_clean()
+
+
+def test_scores_that_grow_from_page_to_page():
+    """The reference of the exponentials has to move several times, by little and by much, up and (in effect) never down, for some heads
+    and not for others, with earlier results rescaled; one to eight CTAs a token."""
+    from rocmforge_b200 import kernels
+    torch.manual_seed(3)
+    T, H, K = 640, 20, 128
+    rows = torch.randn(T, K, device=DEV) * 0.3
+    rows[:, 0] = torch.linspace(-20, 20, T, device=DEV)
+    rows[:, 1] = torch.where(torch.arange(T, device=DEV) % 130 == 77, 30.0, 0.0)
+    q = torch.randn(1, H, K, device=DEV) * 0.3
+    q[0, :, 0] = torch.linspace(-3, 3, H, device=DEV)
+    q[0, ::3, 1] = 2.0
+    rows, q = rows.to(BF16), q.to(BF16)
+    seq, pos, slots, bt, n_pages = _positions([T], [0])
+    pages = torch.zeros(n_pages, 1, 64, K, device=DEV, dtype=BF16)
+    at = bt[slots.long()[seq.long()], (pos // 64).long()].long() * 64 + (pos % 64).long()
+    pages.view(-1, K)[at] = rows
+    want = _softmax_rows(q.double(), rows.double()[:, None], rows.double()[:, None], 1.0, [T - 1])[0]
+    for splits in (1, 2, 4, 8):
+        got = kernels.attention_latent_decode(q, pages, ints([0]), ints([T - 1]), slots, ints([T - 1]), bt, rank=K, scale=1.0, splits=splits)
+        assert (got[0].double() - want).abs().max() < 2e-2 * want.abs().max(), f"{splits} CTAs"
+    status_clean()
+
+
+PREFILL_SIZES = [(4, 32, 16, 32, 64), (5, 48, 24, 96, 136), (3, 128, 64, 128, 512), (2, 16, 8, 144, 40), (2, 80, 0, 16, 64), (3, 64, 40, 112, 320),
+                 (1, 192, 64, 256, 72), (2, 256, 128, 64, 64)]
+
+
+def _expanded(H, D, R, V, K, n, seed):
+    g = torch.Generator(device=DEV).manual_seed(seed)
+    r = lambda *s: torch.randn(*s, generator=g, device=DEV)
+    ld = (K + R + 7) // 8 * 8
+    kv, lat = (r(n, H * (D + V)) * 0.7).to(BF16), (r(n, ld) * 0.7).to(BF16)
+    keys = torch.cat([kv[:, :H * D].double().view(n, H, D), lat[:, K:K + R].double()[:, None].expand(n, H, R)], dim=-1)
+    return kv, lat, keys, kv[:, H * D:].double().view(n, H, V)
+
+
+@pytest.mark.parametrize("gated", [False, True])
+@pytest.mark.parametrize("H,D,R,V,K", PREFILL_SIZES)
+def test_prompts_over_expanded_latents(H, D, R, V, K, gated):
+    """Unequal sequences in one launch, some that start in the middle of a context, query tiles on and off borders of 128 and key
+    tiles on and off borders of 64, against the softmax written out in float64."""
+    from rocmforge_b200 import kernels
+    assert kernels.attention_latent_prefill_supported(H, D, R, V, K)
+    lens, starts = [1, 129, 300, 64, 7], [0, 0, 61, 256, 500]
+    ends = [a + b for a, b in zip(lens, starts)]
+    T, n = sum(lens), sum(ends)
+    kv, lat, keys, vals = _expanded(H, D, R, V, K, n, H + D)
+    torch.manual_seed(D)
+    q = torch.randn(T, H * (D + R) + 16, device=DEV).to(BF16)[:, :H * (D + R)]
+    gate = torch.randn(T, H * V + 8, device=DEV).to(BF16)[:, :H * V] if gated else None
+    tiles = sorted([(i, r) for i, m in enumerate(lens) for r in range(0, m, 128)], key=lambda t: starts[t[0]] + t[1])
+    cu_q, cu_k = [0], [0]
+    for a, e in zip(lens, ends):
+        cu_q.append(cu_q[-1] + a); cu_k.append(cu_k[-1] + e)
+    scale = 1.5 / (D + R) ** 0.5
+    got = kernels.attention_latent_prefill(q, kv, lat, ints(x for t in tiles for x in t), ints(starts), ints(lens), ints(cu_q), ints(cu_k),
+                                           heads=H, dim=D, rot=R, vdim=V, rank=K, scale=scale, gate=gate).double().view(T, H, V)
+    status_clean()
+    for i in range(len(lens)):
+        rows, ctx = slice(cu_q[i], cu_q[i + 1]), slice(cu_k[i], cu_k[i + 1])
+        want = _softmax_rows(q[rows].double().view(-1, H, D + R), keys[ctx], vals[ctx], scale, range(starts[i], ends[i]))
+        if gated:
+            want = want * torch.sigmoid(gate[rows].double()).view(-1, H, V)
+        err = (got[rows] - want).abs().amax(dim=(1, 2))
+        assert err.max() < 2e-2 * max(1.0, float(want.abs().max())), f"sequence {i}, row {int(err.argmax())}"
+
+
+@pytest.mark.parametrize("part", ["unrotated", "rotated"])
+@pytest.mark.parametrize("i,j", [(299, 0), (299, 63), (299, 64), (130, 1), (255, 128), (256, 127), (64, 0), (63, 63), (127, 126), (128, 0)])
+def test_a_far_key_in_a_prompt(i, j, part):
+    """The query at i scores the key at j far above all others, through its unrotated part (one head alone) or through the shared rotated
+    part (all heads), and the key just behind i higher still; whole prompts and a portion that begins at i - 1."""
+    from rocmforge_b200 import kernels
+    H, D, R, V, K, T = 3, 48, 24, 32, 40, 302
+    kv, lat, _, _ = _expanded(H, D, R, V, K, T, i + j)
+    kv, lat = kv.float() * 0.1, lat.float() * 0.1
+    q = torch.randn(T, H, D + R, device=DEV) * 0.1
+    vals = kv[:, H * D:].view(T, H, V)
+    if part == "unrotated":
+        q[i, 1, 0] = 30.0
+        kv[j, D], kv[i + 1, D] = 3.0, 6.0
+        found = [1]
+    else:
+        q[i, :, D] = 30.0
+        lat[j, K], lat[i + 1, K] = 3.0, 6.0
+        found = [0, 1, 2]
+    vals[j], vals[i + 1] = torch.randn(H, V, device=DEV), 1000.0
+    kv, lat, q = kv.to(BF16), lat.to(BF16), q.to(BF16).view(T, -1)
+    for lo in (0, i - 1):
+        n = T - lo
+        tiles = [(0, r) for r in range(0, n, 128)]
+        got = kernels.attention_latent_prefill(q[lo:].contiguous(), kv, lat, ints(x for t in tiles for x in t), ints([lo]), ints([n]), ints([0, n]),
+                                               ints([0, T]), heads=H, dim=D, rot=R, vdim=V, rank=K, scale=1.0).view(n, H, V)
+        want = kv[j, H * D:].view(H, V)
+        for h in found:
+            assert (got[i - lo, h].float() - want[h].float()).abs().max() < 3e-2, f"head {h}, from {lo} on"
+    status_clean()
+
+
+@pytest.mark.parametrize("D,R,V,K", [(576, 0, 576, 8), (600, 40, 700, 8), (1152, 0, 64, 8)])
+def test_the_generic_attention_with_wide_heads(D, R, V, K):
+    """Heads above 512 elements (chunks of 32 keys, a head a pass) against the softmax written out."""
+    from rocmforge_b200 import kernels
+    torch.manual_seed(D)
+    T, H, L = 70, 3, D + R
+    k, v = torch.randn(T, 1, L, device=DEV), torch.randn(T, 1, V, device=DEV)
+    seq, pos, slots, bt, n_pages = _positions([T], [0])
+    at = bt[slots.long()[seq.long()], (pos // 64).long()].long() * 64 + (pos % 64).long()
+    kp, vp = torch.zeros(n_pages, 1, 64, L, device=DEV), torch.zeros(n_pages, 1, 64, V, device=DEV)
+    kp.view(-1, L)[at], vp.view(-1, V)[at] = k[:, 0], v[:, 0]
+    q = torch.randn(T, H, L, device=DEV)
+    got = kernels.attention_generic(q.view(T, H * L), H, 1, L, kp, vp, seq, pos, slots, bt, 0.05, None, v_head_dim=V).view(T, H, V)
+    want = _softmax_rows(q.double(), k.double(), v.double(), 0.05, range(T))
+    assert (got.double() - want).abs().max() < 1e-4
