@@ -130,7 +130,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         }
     } else if (warp == 1) {
         // ---------------- MMA issuer: one thread, accumulator in tensor memory
-        if (lane == 0) {
+        if (elect_one()) {
             constexpr uint32_t idesc = make_idesc(BN);
             bool ok = true;
             for (int i = 0; i < n_kb && ok; ++i) {
