@@ -183,10 +183,19 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
                     const int k_steps = (cnt + 15) >> 4;           // 16 keys each; rows behind the last key are zeroed up to there
                     uint64_t cd = make_smem_desc_mn(smem_u32(c_s) + st * tile_bytes, LD_PAGE_BLOCK);
                     const uint64_t pd = make_smem_desc(smem_u32(p_s) + (vi & 1) * NH * 128);
-                    for (int mb = 0; mb < a.m_blocks; ++mb, cd += (2 * LD_PAGE_BLOCK) >> 4)
-#pragma unroll
-                        for (int ks = 0; ks < 4; ++ks)              // 16 keys = 16 rows of 128 bytes further in C, 32 bytes in P
-                            if (ks < k_steps) tcgen05_mma_bf16(tmem_o + mb * NH, cd + ks * (16 * 128 >> 4), pd + 2 * ks, idesc_o, (vi | ks) ? 1u : 0u);
+                    // a step of 16 keys is 16 rows of 128 bytes further in C and 32 bytes in P
+                    if (k_steps == 4) {
+                        for (int mb = 0; mb < a.m_blocks; ++mb, cd += (2 * LD_PAGE_BLOCK) >> 4) {
+                            tcgen05_mma_bf16(tmem_o + mb * NH, cd, pd, idesc_o, vi ? 1u : 0u);
+                            tcgen05_mma_bf16(tmem_o + mb * NH, cd + 128, pd + 2, idesc_o, 1u);
+                            tcgen05_mma_bf16(tmem_o + mb * NH, cd + 256, pd + 4, idesc_o, 1u);
+                            tcgen05_mma_bf16(tmem_o + mb * NH, cd + 384, pd + 6, idesc_o, 1u);
+                        }
+                    } else {
+                        for (int mb = 0; mb < a.m_blocks; ++mb, cd += (2 * LD_PAGE_BLOCK) >> 4)
+                            for (int ks = 0; ks < k_steps; ++ks)
+                                tcgen05_mma_bf16(tmem_o + mb * NH, cd + 128 * ks, pd + 2 * ks, idesc_o, (vi | ks) ? 1u : 0u);
+                    }
                     tcgen05_commit(b_cfree + 8 * st);
                     tcgen05_commit(b_pvdone + 8 * (vi & 1));
                     ++vi;
@@ -195,10 +204,14 @@ attention_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const 
                     tcgen05_fence_after();
                     uint64_t cd = make_smem_desc(smem_u32(c_s) + (si % a.stages) * tile_bytes), qd = make_smem_desc(smem_u32(q_s));
                     const uint32_t d = tmem_s + (si & 1) * NH;
-                    for (int b = 0; b < a.nb; ++b, cd += LD_PAGE_BLOCK >> 4, qd += (NH * 128) >> 4)
-#pragma unroll
-                        for (int k = 0; k < 4; ++k)
-                            if (4 * b + k < a.n_steps) tcgen05_mma_bf16(d, cd + 2 * k, qd + 2 * k, idesc_s, (b | k) ? 1u : 0u);
+                    const int whole = a.n_steps >> 2;               // blocks of four steps, then the rest of the row
+                    for (int b = 0; b < whole; ++b, cd += LD_PAGE_BLOCK >> 4, qd += (NH * 128) >> 4) {
+                        tcgen05_mma_bf16(d, cd, qd, idesc_s, b ? 1u : 0u);
+                        tcgen05_mma_bf16(d, cd + 2, qd + 2, idesc_s, 1u);
+                        tcgen05_mma_bf16(d, cd + 4, qd + 4, idesc_s, 1u);
+                        tcgen05_mma_bf16(d, cd + 6, qd + 6, idesc_s, 1u);
+                    }
+                    for (int k = 0; k < (a.n_steps & 3); ++k) tcgen05_mma_bf16(d, cd + 2 * k, qd + 2 * k, idesc_s, (whole | k) ? 1u : 0u);
                     tcgen05_commit(b_sfull + 8 * (si & 1));
                     ++si;
                     spin = 0; t0 = 0;
