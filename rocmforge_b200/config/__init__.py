@@ -7,4 +7,5 @@ from .vilulorn import VilulornConfig
 from .figalix import FigalixConfig
 from .ludusun import LudusunConfig
 from .gedilorn import GedilornConfig
+from .dubodra import DubodraConfig
 from . import vilulorn   # (its builder registers "Vilulorn")

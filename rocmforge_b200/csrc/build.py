@@ -37,6 +37,7 @@ MODULES: Dict[str, List[str]] = {
     "moe": ["moe.cu", "common.cuh"],
     "mamba2": ["mamba2.cu", "common.cuh"],
     "mlstm": ["mlstm.cu", "common.cuh"],
+    "layernorm": ["layernorm.cu", "common.cuh"],
     "delta": ["delta.cu", "common.cuh"],
     "streams": ["streams.cu", "common.cuh"],
     "latent": ["latent.cu", "common.cuh"],

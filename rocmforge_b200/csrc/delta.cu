@@ -6,7 +6,7 @@
 //
 //   delta_prepare  q and k heads made unit vectors (x / sqrt(sum x^2 + unit_eps), q also times q_scale), their dot
 //                  products k . q, beta = sigmoid of the projection's columns, and the decays
-//                  g = exp(-exp(A_log_h) softplus(a + dt_bias)) per head and key channel
+//                  g = exp(-exp(A_log_h) softplus(a + dt_bias)) per head and key channel (or one per head)
 //   delta_scan     the recurrence, token by token.  A block owns (sequence, head, 32 value columns): the columns of S are
 //                  independent of each other, so blocks never talk.  Four lanes share a column, each with a quarter of
 //                  its rows in registers over the step's tokens; per token their partial r_k and r_q meet by shuffles.
@@ -18,10 +18,10 @@
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-delta_prepare_kernel(const float* __restrict__ qkv, int qkv_stride, const float* __restrict__ a, const void* __restrict__ dt_bias,
+delta_prepare_kernel(const float* __restrict__ qkv, int qkv_stride, const float* __restrict__ a, int a_stride, const void* __restrict__ dt_bias,
                      const void* __restrict__ a_log, int vec_is_f32, const T* __restrict__ beta_src, int beta_stride,
                      float* __restrict__ qn, float* __restrict__ kn, float* __restrict__ kq, float* __restrict__ decay,
-                     float* __restrict__ beta, int H, int G, int D, float q_scale, float unit_eps) {
+                     float* __restrict__ beta, int H, int G, int D, int per_head, float q_scale, float unit_eps) {
     pdl_trigger();
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
     pdl_wait();
@@ -40,11 +40,12 @@ delta_prepare_kernel(const float* __restrict__ qkv, int qkv_stride, const float*
         }
         if (lane == 0) kq[(size_t)t * G + g] = dot * rq * rk;
     }
-    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H * D; i += gridDim.y * blockDim.x) {
-        const int h = i / D;
-        const float x = a[(size_t)t * H * D + i] + load_vec(dt_bias, vec_is_f32, i);
+    const int ND = per_head ? H : H * D;                 // decays of a token
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < ND; i += gridDim.y * blockDim.x) {
+        const int h = per_head ? i : i / D;
+        const float x = a[(size_t)t * a_stride + i] + load_vec(dt_bias, vec_is_f32, i);
         const float sp = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
-        decay[(size_t)t * H * D + i] = expf(-expf(load_vec(a_log, vec_is_f32, h)) * sp);
+        decay[(size_t)t * ND + i] = expf(-expf(load_vec(a_log, vec_is_f32, h)) * sp);
     }
     for (int h = blockIdx.y * blockDim.x + threadIdx.x; h < H; h += gridDim.y * blockDim.x)
         beta[(size_t)t * H + h] = 1.f / (1.f + expf(-Cvt<T>::to_f32(beta_src[(size_t)t * beta_stride + h])));
@@ -63,7 +64,8 @@ __device__ __forceinline__ void dl_copy4(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-template <int ROWS, int LPC>
+// PER_HEAD: the decay is one number per (token, head) instead of one per key channel.
+template <int ROWS, int LPC, bool PER_HEAD>
 __global__ void __launch_bounds__(DL_WARPS * 32)
 delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ kq,
                   const float* __restrict__ decay, const float* __restrict__ beta, const float* __restrict__ v, int v_stride,
@@ -73,7 +75,8 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
     constexpr int COLS = DL_WARPS * 32 / LPC;                        // value columns of a block
     constexpr int TOK = DP <= 64 ? 16 : (DP <= 128 ? 8 : 4);         // tokens of a stage
     constexpr int NT = DL_WARPS * 32;
-    __shared__ __align__(16) float sk[2][TOK][DP], sq[2][TOK][DP], sg[2][TOK][DP];
+    constexpr int GP = PER_HEAD ? 4 : DP;                            // decays of a token
+    __shared__ __align__(16) float sk[2][TOK][DP], sq[2][TOK][DP], sg[2][TOK][GP];
     __shared__ __align__(16) float sv[2][TOK][COLS];
     __shared__ float sb[2][TOK], skq[2][TOK];
     pdl_trigger();
@@ -88,7 +91,10 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
     // what no copy ever writes: rows beyond dim (k = q = 0, decay 1) and columns beyond vdim (value 0)
     for (int i = tid; i < 2 * TOK * DP; i += NT) {
         const int d = i % DP;
-        if (d >= D) { (&sk[0][0][0])[i] = 0.f; (&sq[0][0][0])[i] = 0.f; (&sg[0][0][0])[i] = 1.f; }
+        if (d >= D) {
+            (&sk[0][0][0])[i] = 0.f; (&sq[0][0][0])[i] = 0.f;
+            if constexpr (!PER_HEAD) (&sg[0][0][0])[i] = 1.f;
+        }
     }
     for (int i = tid; i < 2 * TOK * COLS; i += NT)
         if (j0 + i % COLS >= V) (&sv[0][0][0])[i] = 0.f;
@@ -103,7 +109,7 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
                 const size_t t = (size_t)(t0 + base + tt);
                 dl_copy16(&sk[buf][tt][d], kn + (t * G + hg) * D + d);
                 dl_copy16(&sq[buf][tt][d], qn + (t * G + hg) * D + d);
-                dl_copy16(&sg[buf][tt][d], decay + (t * H + h) * D + d);
+                if constexpr (!PER_HEAD) dl_copy16(&sg[buf][tt][d], decay + (t * H + h) * D + d);
             }
         } else {
             for (int i = tid; i < cnt * D; i += NT) {
@@ -111,7 +117,7 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
                 const size_t t = (size_t)(t0 + base + tt);
                 dl_copy4(&sk[buf][tt][d], kn + (t * G + hg) * D + d);
                 dl_copy4(&sq[buf][tt][d], qn + (t * G + hg) * D + d);
-                dl_copy4(&sg[buf][tt][d], decay + (t * H + h) * D + d);
+                if constexpr (!PER_HEAD) dl_copy4(&sg[buf][tt][d], decay + (t * H + h) * D + d);
             }
         }
         const int nc = min(COLS, V - j0);
@@ -122,6 +128,7 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
         if (tid < cnt) {
             dl_copy4(&sb[buf][tid], beta + (size_t)(t0 + base + tid) * H + h);
             dl_copy4(&skq[buf][tid], kq + (size_t)(t0 + base + tid) * G + hg);
+            if constexpr (PER_HEAD) dl_copy4(&sg[buf][tid][0], decay + (size_t)(t0 + base + tid) * H + h);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -145,7 +152,8 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
         auto fetch = [&](int tt) {
 #pragma unroll
             for (int r = 0; r < ROWS / 4; ++r) {
-                g4[r] = *reinterpret_cast<const float4*>(&sg[buf][tt][rg * 4 + r * 4 * LPC]);
+                if constexpr (PER_HEAD) { const float g = sg[buf][tt][0]; g4[r] = make_float4(g, g, g, g); }
+                else g4[r] = *reinterpret_cast<const float4*>(&sg[buf][tt][rg * 4 + r * 4 * LPC]);
                 k4[r] = *reinterpret_cast<const float4*>(&sk[buf][tt][rg * 4 + r * 4 * LPC]);
                 q4[r] = *reinterpret_cast<const float4*>(&sq[buf][tt][rg * 4 + r * 4 * LPC]);
             }
@@ -185,45 +193,45 @@ delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, co
     }
 }
 
-template <int ROWS, int LPC>
+template <int ROWS, int LPC, bool PER_HEAD>
 static int launch_scan(const float* qn, const float* kn, const float* kq, const float* decay, const float* beta, const float* v,
                        int v_stride, float* state, float* o, const int* cu_q, const int* seq_slot, int B, int H, int G, int D,
                        int V, cudaStream_t st) {
     constexpr int COLS = DL_WARPS * 32 / LPC;
-    rf_launch(delta_scan_kernel<ROWS, LPC>, dim3((V + COLS - 1) / COLS, H, B), dim3(DL_WARPS * 32), 0, st, qn, kn, kq, decay,
+    rf_launch(delta_scan_kernel<ROWS, LPC, PER_HEAD>, dim3((V + COLS - 1) / COLS, H, B), dim3(DL_WARPS * 32), 0, st, qn, kn, kq, decay,
               beta, v, v_stride, state, o, cu_q, seq_slot, H, G, D, V);
     RF_LAUNCH_CHECK();
     return 0;
 }
 
 extern "C" {
-// qkv float [T, qkv_stride]: q heads (G x D), k heads (G x D), then values; a float [T, H*D]; dt_bias [H*D] and a_log [H] of one
-// dtype (vec_is_f32); beta_src [T, beta_stride] of dtype, H columns.  Out: qn, kn float [T, G*D], kq float [T, G], decay float
-// [T, H*D], beta float [T, H].
-int rf_delta_prepare(int dtype, const float* qkv, int qkv_stride, const float* a, const void* dt_bias, const void* a_log,
+// qkv float [T, qkv_stride]: q heads (G x D), k heads (G x D), then values; a float rows of a_stride, H*D columns; dt_bias [H*D]
+// and a_log [H] of one dtype (vec_is_f32); beta_src [T, beta_stride] of dtype, H columns.  Out: qn, kn float [T, G*D], kq float
+// [T, G], decay float [T, H*D], beta float [T, H].  per_head: one decay a head, so a, dt_bias and decay have H columns.
+int rf_delta_prepare(int dtype, const float* qkv, int qkv_stride, const float* a, int a_stride, const void* dt_bias, const void* a_log,
                      int vec_is_f32, const void* beta_src, int beta_stride, float* qn, float* kn, float* kq, float* decay,
-                     float* beta, int H, int G, int D, float q_scale, float unit_eps, int T_, cudaStream_t st) {
+                     float* beta, int H, int G, int D, int per_head, float q_scale, float unit_eps, int T_, cudaStream_t st) {
     if (T_ <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || D <= 0) return RF_ERR_BAD_ARG;
-    int by = T_ >= 512 ? 1 : (H * D + 511) / 512;           // about four decays a thread when there are few tokens
+    int by = T_ >= 512 ? 1 : per_head ? (G + 3) / 4 : (H * D + 511) / 512;           // about four decays a thread when there are few tokens
     if (by > 32) by = 32;
     if (dtype == 0)
-        rf_launch(delta_prepare_kernel<float>, dim3(T_, by), dim3(128), 0, st, qkv, qkv_stride, a, dt_bias, a_log, vec_is_f32,
-                  reinterpret_cast<const float*>(beta_src), beta_stride, qn, kn, kq, decay, beta, H, G, D, q_scale, unit_eps);
+        rf_launch(delta_prepare_kernel<float>, dim3(T_, by), dim3(128), 0, st, qkv, qkv_stride, a, a_stride, dt_bias, a_log, vec_is_f32,
+                  reinterpret_cast<const float*>(beta_src), beta_stride, qn, kn, kq, decay, beta, H, G, D, per_head, q_scale, unit_eps);
     else
-        rf_launch(delta_prepare_kernel<__nv_bfloat16>, dim3(T_, by), dim3(128), 0, st, qkv, qkv_stride, a, dt_bias, a_log, vec_is_f32,
-                  reinterpret_cast<const __nv_bfloat16*>(beta_src), beta_stride, qn, kn, kq, decay, beta, H, G, D, q_scale, unit_eps);
+        rf_launch(delta_prepare_kernel<__nv_bfloat16>, dim3(T_, by), dim3(128), 0, st, qkv, qkv_stride, a, a_stride, dt_bias, a_log, vec_is_f32,
+                  reinterpret_cast<const __nv_bfloat16*>(beta_src), beta_stride, qn, kn, kq, decay, beta, H, G, D, per_head, q_scale, unit_eps);
     RF_LAUNCH_CHECK();
     return 0;
 }
-// state float [slots, H, D, V]; v float [T, v_stride] with head h's values at columns h*V..; o float [T, H*V]; cu_q [B+1]
+// decay float [T, H*D], or (per_head) [T, H]; state float [slots, H, D, V]; v float [T, v_stride] with head h's values at columns h*V..; o float [T, H*V]; cu_q [B+1]
 int rf_delta_scan(const float* qn, const float* kn, const float* kq, const float* decay, const float* beta, const float* v,
                   int v_stride, float* state, float* o, const int* cu_q, const int* seq_slot, int B, int H, int G, int D, int V,
-                  int one_token, int lanes, cudaStream_t st) {
+                  int per_head, int one_token, int lanes, cudaStream_t st) {
     if (B <= 0) return 0;
     if (lanes != 0 && lanes != 4 && lanes != 8) return RF_ERR_BAD_ARG;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || V <= 0 || H > 65535 || B > 65535) return RF_ERR_BAD_ARG;
-#define DL_GO(ROWS, LPC) return launch_scan<ROWS, LPC>(qn, kn, kq, decay, beta, v, v_stride, state, o, cu_q, seq_slot, B, H, G, D, V, st)
+#define DL_GO(ROWS, LPC) return (per_head ? launch_scan<ROWS, LPC, true> : launch_scan<ROWS, LPC, false>)(qn, kn, kq, decay, beta, v, v_stride, state, o, cu_q, seq_slot, B, H, G, D, V, st)
     // Steps of one token a sequence (the state is read and written once, nothing else): four lanes a column.  Steps with
     // longer portions: eight lanes a column (twice the blocks, half the chain of each; fetching the next token's operands
     // into registers ahead of the chain was measured and cost more in registers than it hid).  The two forms add a column's products in another order: a difference of rounding between a token

@@ -462,8 +462,8 @@ rope_kv_write_rows_kernel(const T* __restrict__ src, int row_stride, T* __restri
 
 // ---------------------------------------------------------------- SwiGLU
 // gu: [T, 2I] with gate_j at column 2j and up_j at column 2j+1 (the fused weight is
-// interleaved row by row at load time); a[t, j] = silu(gate) * up (RELU: relu(gate) * up), evaluated in 32-bit.
-template <typename T, bool RELU>
+// interleaved row by row at load time); a[t, j] = act(gate) * up, evaluated in 32-bit; ACT 0: silu, 1: relu, 2: gelu by tanh.
+template <typename T, int ACT>
 __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ a, size_t n_out, int I) {
     pdl_trigger();
     pdl_wait();
@@ -472,7 +472,11 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ a, size_
         const size_t t = idx / I, j = idx - t * I;
         const float g = Cvt<T>::to_f32(gu[t * 2 * I + 2 * j]);
         const float u = Cvt<T>::to_f32(gu[t * 2 * I + 2 * j + 1]);
-        a[idx] = Cvt<T>::from_f32((RELU ? fmaxf(g, 0.f) : g / (1.f + expf(-g))) * u);
+        float act;
+        if constexpr (ACT == 0) act = g / (1.f + expf(-g));
+        else if constexpr (ACT == 1) act = fmaxf(g, 0.f);
+        else act = 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+        a[idx] = Cvt<T>::from_f32(act * u);
     }
 }
 
@@ -1075,12 +1079,12 @@ static int launch_rope_kv_write(const void* src, int row_stride, int n_partials,
     return 0;
 }
 
-template <typename T, bool RELU = false>
+template <typename T, int ACT = 0>
 static int launch_swiglu(const void* gu, void* a, int T_, int I, cudaStream_t st) {
     const size_t n = (size_t)T_ * I;
     if (n == 0) return 0;
     const int blocks = (int)((n + 255) / 256 > 148 * 16 ? 148 * 16 : (n + 255) / 256);
-    rf_launch(swiglu_kernel<T, RELU>, dim3(blocks), dim3(256), 0, st, reinterpret_cast<const T*>(gu), reinterpret_cast<T*>(a), n, I);
+    rf_launch(swiglu_kernel<T, ACT>, dim3(blocks), dim3(256), 0, st, reinterpret_cast<const T*>(gu), reinterpret_cast<T*>(a), n, I);
     RF_LAUNCH_CHECK();
     return 0;
 }
@@ -1201,7 +1205,10 @@ int rf_swiglu(int dtype, const void* gu, void* a, int T_, int I, cudaStream_t st
     return dtype == 0 ? launch_swiglu<float>(gu, a, T_, I, st) : launch_swiglu<__nv_bfloat16>(gu, a, T_, I, st);
 }
 int rf_reglu(int dtype, const void* gu, void* a, int T_, int I, cudaStream_t st) {
-    return dtype == 0 ? launch_swiglu<float, true>(gu, a, T_, I, st) : launch_swiglu<__nv_bfloat16, true>(gu, a, T_, I, st);
+    return dtype == 0 ? launch_swiglu<float, 1>(gu, a, T_, I, st) : launch_swiglu<__nv_bfloat16, 1>(gu, a, T_, I, st);
+}
+int rf_geglu(int dtype, const void* gu, void* a, int T_, int I, cudaStream_t st) {
+    return dtype == 0 ? launch_swiglu<float, 2>(gu, a, T_, I, st) : launch_swiglu<__nv_bfloat16, 2>(gu, a, T_, I, st);
 }
 int rf_relu2(int dtype, const void* x, void* a, long long n, cudaStream_t st) {
     return dtype == 0 ? launch_relu2<float>(x, a, n, st) : launch_relu2<__nv_bfloat16>(x, a, n, st);

@@ -11,7 +11,8 @@
 // across CTAs (grid.z), each split writing its own 32-bit partial sums, which the next
 // add+RMSNorm kernel adds in index order (no atomics: the result never depends on timing).
 // Epilogues: + bias, 32-bit output, accumulate into the 32-bit residual stream, and the
-// units silu(gate) * up (SWIGLU) and relu(gate) * up (REGLU) on row-interleaved gate/up weights.
+// units silu(gate) * up (SWIGLU), relu(gate) * up (REGLU), gelu(gate) * up (GEGLU) and the one with clamped halves (CLAMPGLU) on
+// row-interleaved gate/up weights.
 //
 // maeddesg/ROCmForge's counterparts are its RDNA-WMMA prefill GEMMs (hip_kernels/wmma/
 // wmma_gemm_tiled.hip:57-195: 64x64x16 tiles, FP16 operands, FP32 accumulate) and its decode
@@ -209,17 +210,19 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                                 reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.ldo + (n >> 1)] =
                                     __float2bfloat16_rn(silu_fast(g) * u);
                         }
-                    } else if (p.mode == EPI_REGLU) {    // the same exchange, relu instead of silu
+                    } else if (epi_gated(p.mode)) {      // the same exchange for another unit
                         const bool odd = lane & 1;
+                        with_gated_unit(p.mode, p.limit, p.alpha, [&](auto unit) {
 #pragma unroll
-                        for (int j = 0; j < CH; j += 2) {
-                            const float v0 = __uint_as_float(r[j]) + b, v1 = __uint_as_float(r[j + 1]) + b;
-                            const float got = __shfl_xor_sync(0xffffffffu, odd ? v0 : v1, 1);
-                            const float g = odd ? got : v0, u = odd ? v1 : got;
-                            const int m = m0 + j + (odd ? 1 : 0);
-                            if (m < p.M && (n | 1) < p.N)
-                                reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.ldo + (n >> 1)] = __float2bfloat16_rn(fmaxf(g, 0.f) * u);
-                        }
+                            for (int j = 0; j < CH; j += 2) {
+                                const float v0 = __uint_as_float(r[j]) + b, v1 = __uint_as_float(r[j + 1]) + b;
+                                const float got = __shfl_xor_sync(0xffffffffu, odd ? v0 : v1, 1);
+                                const float g = odd ? got : v0, u = odd ? v1 : got;
+                                const int m = m0 + j + (odd ? 1 : 0);
+                                if (m < p.M && (n | 1) < p.N)
+                                    reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.ldo + (n >> 1)] = __float2bfloat16_rn(unit(g, u));
+                            }
+                        });
                     } else if (n < p.N) {
                         // the mode, the output's base and the number of tokens that exist are settled once per chunk: a
                         // token then costs an add and a store (settling them per element made a chunk of 32 tokens take
@@ -377,17 +380,16 @@ extern "C" {
 int rf_gemm_tc_supported(int M, int N, int K, int mode) {
     if (M <= 0 || N <= 0 || K <= 0) return 0;
     if (K % 8) return 0;                              // TMA needs 16-byte row strides
-    if ((mode == EPI_SWIGLU || mode == EPI_CLAMPGLU || mode == EPI_REGLU) && (N % 2)) return 0;
+    if (epi_gated(mode) && (N % 2)) return 0;
     return encode_fn() != nullptr;
 }
 
-// Tokens as rows: out[M, N] (mode STORE / F32 / RESIDUAL) or out[M, N/2] (SWIGLU, REGLU).
-int rf_gemm_tc(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo,
-               int M, int N, int K, int mode, int* status, cudaStream_t st) {
+static int gemm_rows(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo, int M, int N,
+                     int K, int mode, float limit, float alpha, int* status, cudaStream_t st) {
     if (!rf_gemm_tc_supported(M, N, K, mode) || mode == EPI_PARTIAL || mode == EPI_RESNORM) return RF_ERR_UNSUPPORTED;
     CUtensorMap ma, mb;
     int e;
-    TcParams p{out, bias, bias_is_f32, M, N, K, ldo, mode, (K + TC_BK - 1) / TC_BK, 0, status, 1};
+    TcParams p{out, bias, bias_is_f32, M, N, K, ldo, mode, (K + TC_BK - 1) / TC_BK, limit, 0, status, 1, alpha};
     if (N > 128) {
         if ((e = make_map(&ma, X, M, K, ldx, TC_BM)) || (e = make_map(&mb, W, N, K, K, 256))) return e;
         dim3 grid((N + 255) / 256, (M + TC_BM - 1) / TC_BM, 1);
@@ -396,6 +398,18 @@ int rf_gemm_tc(const void* X, int ldx, const void* W, const void* bias, int bias
     if ((e = make_map(&ma, X, M, K, ldx, TC_BM)) || (e = make_map(&mb, W, N, K, K, 128))) return e;
     dim3 grid((N + 127) / 128, (M + TC_BM - 1) / TC_BM, 1);
     return launch_cfg<128, false, 6>(ma, mb, p, grid, st);
+}
+
+// Tokens as rows: out[M, N] (mode STORE / F32 / RESIDUAL) or out[M, N/2] (SWIGLU, REGLU, GEGLU).
+int rf_gemm_tc(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo,
+               int M, int N, int K, int mode, int* status, cudaStream_t st) {
+    if (mode == EPI_CLAMPGLU) return RF_ERR_BAD_ARG;              // that mode comes with its constants, below
+    return gemm_rows(X, ldx, W, bias, bias_is_f32, out, ldo, M, N, K, mode, 0.f, 0.f, status, st);
+}
+// Mode CLAMPGLU: out[M, N/2] = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit).
+int rf_gemm_tc_glu(const void* X, int ldx, const void* W, void* out, int ldo, int M, int N, int K, float limit, float alpha,
+                   int* status, cudaStream_t st) {
+    return gemm_rows(X, ldx, W, nullptr, 0, out, ldo, M, N, K, EPI_CLAMPGLU, limit, alpha, status, st);
 }
 
 // Many weight matrices in one launch (see GROUPED above): X [n_rows, K] holds the rows sorted by group, W [groups, N, K]
@@ -411,7 +425,7 @@ static int gemm_tc_grouped(const void* X, int ldx, int n_rows, const void* W, in
     if (max_tiles > 65535) return RF_ERR_UNSUPPORTED;
     CUtensorMap ma, mb;
     int e;
-    TcParams p{out, nullptr, 0, n_rows, N, K, ldo, mode, (K + TC_BK - 1) / TC_BK, 0, status, 1};
+    TcParams p{out, nullptr, 0, n_rows, N, K, ldo, mode, (K + TC_BK - 1) / TC_BK, 0.f, 0, status, 1, 0.f};
     const TcGroup grp{tiles, N, row_scale, limit, alpha};
     if (N > 128) {
         if ((e = make_map(&ma, X, n_rows, K, ldx, TC_BM)) || (e = make_map(&mb, W, (long long)groups * N, K, K, 256))) return e;
@@ -444,10 +458,10 @@ int rf_gemm_tc_grouped_glu(const void* X, int ldx, int n_rows, const void* W, in
 // Mode RESNORM (splits = 1, 2, 4 or 8: the splits of an output tile are one thread-block cluster and add their
 // partial sums through each other's shared memory): resid [M, N] += the product (+ bias), normed [M, N] = resid *
 // norm_w in bfloat16, ss_out [ceil(N/128)][ss_out_stride] = each weight tile's sum of resid^2 per token; out is not used.
-int rf_gemm_tc_skinny_ex(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo,
+static int gemm_skinny(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo,
                          int M, int N, int K, int mode, int splits, const float* ss_in, int ss_in_tiles,
                          int ss_in_stride, float ss_eps, float* resid, const void* norm_w, int norm_w_is_f32,
-                         void* normed, float* ss_out, int ss_out_stride, int* status, cudaStream_t st) {
+                         void* normed, float* ss_out, int ss_out_stride, float limit, float alpha, int* status, cudaStream_t st) {
     if (!rf_gemm_tc_supported(M, N, K, mode) || M > 256 || splits < 1) return RF_ERR_UNSUPPORTED;
     if (splits > 1 && mode != EPI_PARTIAL && mode != EPI_RESNORM) return RF_ERR_BAD_ARG;
     if (mode == EPI_RESNORM && (!resid || !norm_w || !normed || !ss_out || ldo != N || ss_out_stride < M))
@@ -458,7 +472,7 @@ int rf_gemm_tc_skinny_ex(const void* X, int ldx, const void* W, const void* bias
     const int kb = (K + TC_BK - 1) / TC_BK;
     const int per = (kb + splits - 1) / splits;
     if ((splits - 1) * per >= kb) return RF_ERR_BAD_ARG;          // an empty split would leave its partial unwritten
-    TcParams p{mode == EPI_RESNORM ? (void*)resid : out, bias, bias_is_f32, M, N, K, ldo, mode, per, (long long)M * ldo, status, 1};
+    TcParams p{mode == EPI_RESNORM ? (void*)resid : out, bias, bias_is_f32, M, N, K, ldo, mode, per, limit, (long long)M * ldo, status, 1, alpha};
     const TcNorm nrm = TcNorm{norm_w, reinterpret_cast<__nv_bfloat16*>(normed), ss_out, ss_in, norm_w_is_f32, ss_out_stride,
                               ss_in_tiles, ss_in_stride, ss_eps, 1.0f / (float)K};
     static_assert(sizeof(TcParams) + sizeof(TcNorm) <= 128, "two tensor maps and these must stay within 384 bytes");
@@ -484,6 +498,21 @@ int rf_gemm_tc_skinny_ex(const void* X, int ldx, const void* W, const void* bias
     if (bn == 32) return launch_cfg<32, true, 5>(ma, mb, p, grid, st);
     if (bn == 64) return launch_cfg<64, true, 4>(ma, mb, p, grid, st);
     return launch_cfg<128, true, 3>(ma, mb, p, grid, st);
+}
+
+int rf_gemm_tc_skinny_ex(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo,
+                         int M, int N, int K, int mode, int splits, const float* ss_in, int ss_in_tiles,
+                         int ss_in_stride, float ss_eps, float* resid, const void* norm_w, int norm_w_is_f32,
+                         void* normed, float* ss_out, int ss_out_stride, int* status, cudaStream_t st) {
+    if (mode == EPI_CLAMPGLU) return RF_ERR_BAD_ARG;              // that mode comes with its constants, below
+    return gemm_skinny(X, ldx, W, bias, bias_is_f32, out, ldo, M, N, K, mode, splits, ss_in, ss_in_tiles, ss_in_stride, ss_eps,
+                       resid, norm_w, norm_w_is_f32, normed, ss_out, ss_out_stride, 0.f, 0.f, status, st);
+}
+// Mode CLAMPGLU (see rf_gemm_tc_glu) for few tokens.
+int rf_gemm_tc_skinny_glu(const void* X, int ldx, const void* W, void* out, int ldo, int M, int N, int K, const float* ss_in,
+                          int ss_in_tiles, int ss_in_stride, float ss_eps, float limit, float alpha, int* status, cudaStream_t st) {
+    return gemm_skinny(X, ldx, W, nullptr, 0, out, ldo, M, N, K, EPI_CLAMPGLU, 1, ss_in, ss_in_tiles, ss_in_stride, ss_eps,
+                       nullptr, nullptr, 0, nullptr, nullptr, 0, limit, alpha, status, st);
 }
 
 int rf_gemm_tc_skinny(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo,

@@ -311,20 +311,22 @@ gemm_tc_cluster_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_c
                 }
                 const uint32_t srow = smem_u32(st) + row * 128;
                 const int n0 = tile_n * bn + c;
-                if (mode == EPI_REGLU) {             // 32 accumulators -> 16 bfloat16 = 2 chunks of 16 bytes
+                if (epi_gated(mode) && mode != EPI_SWIGLU) {     // 32 accumulators -> 16 bfloat16 = 2 chunks of 16 bytes
+                    with_gated_unit(mode, p.limit, p.alpha, [&](auto unit) {
 #pragma unroll
-                    for (int h8 = 0; h8 < 2; ++h8) {
-                        uint32_t wv[4];
+                        for (int h8 = 0; h8 < 2; ++h8) {
+                            uint32_t wv[4];
 #pragma unroll
-                        for (int q = 0; q < 4; ++q) {
-                            const int j = h8 * 16 + 4 * q;
-                            wv[q] = pack_bf16x2(fmaxf(__uint_as_float(r[j]), 0.f) * __uint_as_float(r[j + 1]),
-                                                fmaxf(__uint_as_float(r[j + 2]), 0.f) * __uint_as_float(r[j + 3]));
+                            for (int q = 0; q < 4; ++q) {
+                                const int j = h8 * 16 + 4 * q;
+                                wv[q] = pack_bf16x2(unit(__uint_as_float(r[j]), __uint_as_float(r[j + 1])),
+                                                    unit(__uint_as_float(r[j + 2]), __uint_as_float(r[j + 3])));
+                            }
+                            const int chunk = (cc >> 4) + h8;
+                            asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(srow + ((chunk ^ (row & 7)) << 4)),
+                                         "r"(wv[0]), "r"(wv[1]), "r"(wv[2]), "r"(wv[3]) : "memory");
                         }
-                        const int chunk = (cc >> 4) + h8;
-                        asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(srow + ((chunk ^ (row & 7)) << 4)),
-                                     "r"(wv[0]), "r"(wv[1]), "r"(wv[2]), "r"(wv[3]) : "memory");
-                    }
+                    });
                 } else if (mode == EPI_SWIGLU) {     // the same with silu
 #pragma unroll
                     for (int h8 = 0; h8 < 2; ++h8) {
@@ -365,7 +367,7 @@ gemm_tc_cluster_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_c
                 epi_barrier();
                 if (leader) {
                     // output column of the slab's first element, in elements of the output matrix
-                    const int oc0 = (mode == EPI_SWIGLU || mode == EPI_REGLU) ? (tile_n * bn + c0) / 2 : tile_n * bn + c0;
+                    const int oc0 = epi_gated(mode) ? (tile_n * bn + c0) / 2 : tile_n * bn + c0;
                     if (!ordered) {                      // the tile's earlier K parts must have been added
                         unsigned long long t0 = 0;
                         for (long long spin = 0; !abort_flag; ++spin) {
@@ -539,7 +541,7 @@ static int launch_cluster(const void* X, int ldx, const void* W, TcParams p, int
     int e;
     if ((e = make_map(&ma, X, p.M, p.K, ldx, TC_BM)) || (e = make_map(&mb, W, p.N, p.K, p.K, bn / CL))) return e;
     const bool f32_out = p.mode == EPI_F32 || p.mode == EPI_RESIDUAL;
-    const long long out_cols = (p.mode == EPI_SWIGLU || p.mode == EPI_REGLU) ? p.N / 2 : p.N;
+    const long long out_cols = epi_gated(p.mode) ? p.N / 2 : p.N;
     if ((e = make_out_map(&mo, p.out, p.M, out_cols, p.ldo, f32_out))) return e;
     const int tiles_n = (p.N + bn - 1) / bn;
     int n_clusters = groups_m * tiles_n * p.splits;
@@ -564,9 +566,9 @@ int rf_gemm_tc_cluster_supported(int M, int N, int K, int mode) {
     // more tokens than the skinny kernel takes: below 256 rows a cluster's second CTA works on an empty tile, which
     // still beats 14 unclustered CTAs streaming a 3,584-row weight (decode at batch 128: 8.0 ms a step without)
     if (M <= 64 || N < CG_BN || K <= 0 || K % 8) return 0;
-    if ((mode == EPI_SWIGLU || mode == EPI_REGLU) && (N % 2)) return 0;
+    if (epi_gated(mode) && (N % 2)) return 0;
     if (mode == EPI_PARTIAL) return 0;
-    const int out_cols = (mode == EPI_SWIGLU || mode == EPI_REGLU) ? N / 2 : N;
+    const int out_cols = epi_gated(mode) ? N / 2 : N;
     if (out_cols % 8) return 0;                      // TMA stores need 16-byte row strides
     return encode_fn() != nullptr;
 }
@@ -577,16 +579,27 @@ int rf_gemm_tc_cluster_supported(int M, int N, int K, int mode) {
 // How many clusters of `cluster` CTAs run at once (what the persistent grid is sized to), or a negative code.
 int rf_gemm_tc_cluster_width(int cluster);
 
-int rf_gemm_tc_cluster(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo,
-                       int M, int N, int K, int mode, int cluster, int parts, int* flags, int n_flags, int* status,
-                       cudaStream_t st) {
+static int gemm_cluster(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo, int M, int N,
+                        int K, int mode, int cluster, int parts, int* flags, int n_flags, float limit, float alpha, int* status,
+                        cudaStream_t st) {
     if (!rf_gemm_tc_cluster_supported(M, N, K, mode)) return RF_ERR_UNSUPPORTED;
     if (parts < 0 || parts > 5) return RF_ERR_BAD_ARG;
-    TcParams p{out, bias, bias_is_f32, M, N, K, ldo, mode, (K + TC_BK - 1) / TC_BK, 0, status, 1};
+    TcParams p{out, bias, bias_is_f32, M, N, K, ldo, mode, (K + TC_BK - 1) / TC_BK, limit, 0, status, 1, alpha};
     if (cluster == 2 && g_pair) return launch_cluster<2, true>(X, ldx, W, p, parts, flags, n_flags, st);
     if (cluster == 2) return launch_cluster<2, false>(X, ldx, W, p, parts, flags, n_flags, st);
     if (cluster == 4) return launch_cluster<4, false>(X, ldx, W, p, parts, flags, n_flags, st);
     return RF_ERR_BAD_ARG;
+}
+int rf_gemm_tc_cluster(const void* X, int ldx, const void* W, const void* bias, int bias_is_f32, void* out, int ldo,
+                       int M, int N, int K, int mode, int cluster, int parts, int* flags, int n_flags, int* status,
+                       cudaStream_t st) {
+    if (mode == EPI_CLAMPGLU) return RF_ERR_BAD_ARG;              // that mode comes with its constants, below
+    return gemm_cluster(X, ldx, W, bias, bias_is_f32, out, ldo, M, N, K, mode, cluster, parts, flags, n_flags, 0.f, 0.f, status, st);
+}
+// Mode CLAMPGLU: out[M, N/2] = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit).
+int rf_gemm_tc_cluster_glu(const void* X, int ldx, const void* W, void* out, int ldo, int M, int N, int K, int cluster, float limit,
+                           float alpha, int* status, cudaStream_t st) {
+    return gemm_cluster(X, ldx, W, nullptr, 0, out, ldo, M, N, K, EPI_CLAMPGLU, cluster, 0, nullptr, 0, limit, alpha, status, st);
 }
 
 int rf_gemm_tc_cluster_width(int cluster) {

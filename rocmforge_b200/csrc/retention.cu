@@ -13,6 +13,7 @@
 //                       column; a lane holds the rows lane, lane + 32, ... of it in registers.  The order of every sum
 //                       is fixed by (dim, position in the sequence) alone: how a prompt is cut into steps, or what
 //                       else is in the batch, changes no bit.
+//   silu_columns, row_norm_gate   for designs whose q, k and v pass silu and whose heads are normed together (below)
 //   retention_gate      o / rms(o) per head, times silu(gate), into the compute dtype for the output product
 #include "common.cuh"
 
@@ -57,10 +58,77 @@ __global__ void retention_prepare_kernel(const T* __restrict__ src, int row_stri
     }
 }
 
+// out[t, c] = silu(src[t, c]) as float [T, W]: the inputs of a recurrence whose q, k and v pass silu.  src is the product's
+// matrix (n_partials 0) or its partial sums, added in index order.  Four columns a thread (W a multiple of 4) or one.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+silu_columns_kernel(const void* __restrict__ src, int n_partials, long long part_stride, int row_stride, float* __restrict__ out,
+                    int W, size_t n) {
+    pdl_trigger();
+    pdl_wait();
+    const int per_row = W / V;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = i / per_row;
+        const int c = (int)(i - t * per_row) * V;
+        float x[V];
+#pragma unroll
+        for (int u = 0; u < V; ++u) x[u] = 0.f;
+        if (n_partials > 0) {
+            const float* p = reinterpret_cast<const float*>(src) + t * row_stride + c;
+#pragma unroll 8
+            for (int s = 0; s < n_partials; ++s) {
+                if constexpr (V == 4) {
+                    const float4 a = *reinterpret_cast<const float4*>(p + (size_t)s * part_stride);
+                    x[0] += a.x; x[1] += a.y; x[2] += a.z; x[3] += a.w;
+                } else x[0] += p[(size_t)s * part_stride];
+            }
+        } else {
+            alignas(16) T v[V];
+            const T* p = reinterpret_cast<const T*>(src) + t * row_stride + c;
+            if constexpr (V == 4 && sizeof(T) == 2) *reinterpret_cast<uint2*>(v) = *reinterpret_cast<const uint2*>(p);
+            else if constexpr (V == 4) *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(p);
+            else v[0] = *p;
+#pragma unroll
+            for (int u = 0; u < V; ++u) x[u] = Cvt<T>::to_f32(v[u]);
+        }
+#pragma unroll
+        for (int u = 0; u < V; ++u) x[u] = x[u] / (1.f + expf(-x[u]));
+        if constexpr (V == 4) *reinterpret_cast<float4*>(out + t * W + c) = make_float4(x[0], x[1], x[2], x[3]);
+        else out[t * W + c] = x[0];
+    }
+}
+
+// A block per token: o / sqrt(mean(o^2) + eps) over the whole row (all heads together), times a weight [W], times
+// sigmoid(gate) or silu(gate), in the compute dtype.  The gate comes in the compute dtype, or as partial sums.
+template <typename T>
+__global__ void __launch_bounds__(1024)
+row_norm_gate_kernel(const float* __restrict__ o, const void* __restrict__ gate, int n_partials, long long part_stride,
+                     int gate_stride, T* __restrict__ out, int W, float eps, const void* __restrict__ norm_w, int w_is_f32,
+                     int sigmoid) {
+    __shared__ float red[34];
+    pdl_trigger();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const float* orow = o + t * W;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += blockDim.x) { const float x = orow[c]; ss += x * x; }
+    const float r = rsqrtf(block_sum(ss, red) / (float)W + eps);
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+        float g = 0.f;
+        if (n_partials > 0) {
+            const float* p = reinterpret_cast<const float*>(gate) + t * gate_stride + c;
+#pragma unroll 8
+            for (int s = 0; s < n_partials; ++s) g += p[(size_t)s * part_stride];
+        } else g = Cvt<T>::to_f32(reinterpret_cast<const T*>(gate)[t * gate_stride + c]);
+        const float gv = (sigmoid ? 1.f : g) / (1.f + expf(-g));
+        out[t * W + c] = Cvt<T>::from_f32(orow[c] * r * load_vec(norm_w, w_is_f32, c) * gv);
+    }
+}
+
 // grid (sequence, head, ceil(vdim / RT_COLS)); block RT_COLS warps.  R = ceil(dim / 32) rows of a column per lane.
 template <typename T, int R>
 __global__ void __launch_bounds__(RT_COLS * 32)
-retention_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const T* __restrict__ v, int v_stride,
+retention_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, int qk_stride, const T* __restrict__ v, int v_stride,
                       float* __restrict__ state, const float* __restrict__ decay, float* __restrict__ o,
                       const int* __restrict__ cu_q, const int* __restrict__ seq_slot, int heads, int dim, int vdim) {
     extern __shared__ float sh[];                     // q [RT_TOK][dim], k [RT_TOK][dim], v [RT_TOK][RT_COLS]
@@ -74,7 +142,6 @@ retention_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, 
     const int row0 = cu_q[b], row1 = cu_q[b + 1];
     const int slot = seq_slot[b];
     const float d = decay[h];
-    const int width = heads * dim;
     float* S = state + (((size_t)slot * heads + h) * vdim + (j < vdim ? j : 0)) * dim;      // this warp's column
     pdl_wait();
     float s[R];
@@ -88,8 +155,8 @@ retention_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, 
         __syncthreads();                              // the tokens before are used up
         for (int idx = threadIdx.x; idx < cnt * dim; idx += blockDim.x) {
             const int tt = idx / dim, i = idx - tt * dim;
-            qs[idx] = q[(size_t)(t0 + tt) * width + h * dim + i];
-            ks[idx] = k[(size_t)(t0 + tt) * width + h * dim + i];
+            qs[idx] = q[(size_t)(t0 + tt) * qk_stride + h * dim + i];
+            ks[idx] = k[(size_t)(t0 + tt) * qk_stride + h * dim + i];
         }
         for (int idx = threadIdx.x; idx < cnt * RT_COLS; idx += blockDim.x) {
             const int tt = idx / RT_COLS, c = idx - tt * RT_COLS;
@@ -167,7 +234,7 @@ __global__ void retention_gate_kernel(const float* __restrict__ o, const T* __re
 // by dim) and columns 4 tx .. 4 tx + 3: per key, 16-byte loads of its k rows and of its v columns feed 4 RPT FMAs
 template <typename T>
 __global__ void __launch_bounds__(256)
-retention_chunk_state_kernel(const float* __restrict__ k, const T* __restrict__ v, int v_stride, float* __restrict__ LS,
+retention_chunk_state_kernel(const float* __restrict__ k, int qk_stride, const T* __restrict__ v, int v_stride, float* __restrict__ LS,
                              const float* __restrict__ decay, const int* __restrict__ table, const int* __restrict__ cu_q,
                              int B, int heads, int dim, int vdim) {
     extern __shared__ __align__(16) float sh[];
@@ -179,13 +246,12 @@ retention_chunk_state_kernel(const float* __restrict__ k, const T* __restrict__ 
     const int c = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * RV;
     const int b = table[B + 1 + 2 * c], q0 = table[B + 2 + 2 * c];
     const int row0 = cu_q[b] + q0, cnt = min(RC, cu_q[b + 1] - row0);
-    const int width = heads * dim;
     if (threadIdx.x < RC) pw[threadIdx.x] = powf(decay[h], (float)threadIdx.x);
     pdl_wait();
     __syncthreads();
     for (int idx = threadIdx.x; idx < cnt * dimP; idx += 256) {
         const int s = idx / dimP, i = idx - s * dimP;
-        ks[idx] = i < dim ? k[(size_t)(row0 + s) * width + h * dim + i] * pw[cnt - 1 - s] : 0.f;
+        ks[idx] = i < dim ? k[(size_t)(row0 + s) * qk_stride + h * dim + i] * pw[cnt - 1 - s] : 0.f;
     }
     for (int idx = threadIdx.x; idx < cnt * RV; idx += 256) {
         const int s = idx / RV, j = idx - s * RV;
@@ -261,7 +327,7 @@ retention_chunk_carry_kernel(float* __restrict__ LS, float* __restrict__ state, 
 // grid (chunk, head, ceil(vdim / RV)); 256 threads as a 16 x 16 grid of 4 x 4 tiles
 template <typename T>
 __global__ void __launch_bounds__(256)
-retention_chunk_out_kernel(const float* __restrict__ q, const float* __restrict__ k, const T* __restrict__ v, int v_stride,
+retention_chunk_out_kernel(const float* __restrict__ q, const float* __restrict__ k, int qk_stride, const T* __restrict__ v, int v_stride,
                            const float* __restrict__ LS, const float* __restrict__ decay, float* __restrict__ o,
                            const int* __restrict__ table, const int* __restrict__ cu_q, int B, int heads, int dim, int vdim) {
     extern __shared__ __align__(16) float sh[];
@@ -275,14 +341,13 @@ retention_chunk_out_kernel(const float* __restrict__ q, const float* __restrict_
     const int b = table[B + 1 + 2 * c], q0 = table[B + 2 + 2 * c];
     const int row0 = cu_q[b] + q0, cnt = min(RC, cu_q[b + 1] - row0);
     const float d = decay[h];
-    const int width = heads * dim;
     if (threadIdx.x <= RC) pw[threadIdx.x] = powf(d, (float)threadIdx.x);
     pdl_wait();
     for (int idx = threadIdx.x; idx < RC * dim; idx += 256) {
         const int s = idx / dim, i = idx - s * dim;
         const bool in = s < cnt;
-        qt[i * RC_LD + s] = in ? q[(size_t)(row0 + s) * width + h * dim + i] : 0.f;
-        kt[i * RC_LD + s] = in ? k[(size_t)(row0 + s) * width + h * dim + i] : 0.f;
+        qt[i * RC_LD + s] = in ? q[(size_t)(row0 + s) * qk_stride + h * dim + i] : 0.f;
+        kt[i * RC_LD + s] = in ? k[(size_t)(row0 + s) * qk_stride + h * dim + i] : 0.f;
     }
     for (int idx = threadIdx.x; idx < RC * RV; idx += 256) {
         const int s = idx / RV, j = idx - s * RV;
@@ -358,7 +423,7 @@ retention_chunk_out_kernel(const float* __restrict__ q, const float* __restrict_
 }
 
 template <typename T>
-static int launch_chunked(const float* q, const float* k, const void* v, int v_stride, float* state, const float* decay,
+static int launch_chunked(const float* q, const float* k, int qk_stride, const void* v, int v_stride, float* state, const float* decay,
                           float* o, float* LS, const int* table, int n_chunks, const int* cu_q, const int* seq_slot, int B,
                           int heads, int dim, int vdim, cudaStream_t st) {
     if (B <= 0 || n_chunks <= 0) return 0;
@@ -377,13 +442,13 @@ static int launch_chunked(const float* q, const float* k, const void* v, int v_s
         if (e != cudaSuccess) return (int)e;
         set3 = smem3;
     }
-    rf_launch(retention_chunk_state_kernel<T>, dim3(n_chunks, heads, vz), dim3(256), smem1, st, k, reinterpret_cast<const T*>(v),
+    rf_launch(retention_chunk_state_kernel<T>, dim3(n_chunks, heads, vz), dim3(256), smem1, st, k, qk_stride, reinterpret_cast<const T*>(v),
               v_stride, LS, decay, table, cu_q, B, heads, dim, vdim);
     RF_LAUNCH_CHECK();
     rf_launch(retention_chunk_carry_kernel, dim3(B, heads, (dim * vdim + 255) / 256), dim3(256), 0, st, LS, state, decay, table,
               cu_q, seq_slot, heads, dim, vdim);
     RF_LAUNCH_CHECK();
-    rf_launch(retention_chunk_out_kernel<T>, dim3(n_chunks, heads, vz), dim3(256), smem3, st, q, k, reinterpret_cast<const T*>(v),
+    rf_launch(retention_chunk_out_kernel<T>, dim3(n_chunks, heads, vz), dim3(256), smem3, st, q, k, qk_stride, reinterpret_cast<const T*>(v),
               v_stride, (const float*)LS, decay, o, table, cu_q, B, heads, dim, vdim);
     RF_LAUNCH_CHECK();
     return 0;
@@ -404,29 +469,29 @@ static int launch_prepare(const void* src, int row_stride, int q_col, int k_col,
 }
 
 template <typename T, int R>
-static int launch_scan_r(const float* q, const float* k, const void* v, int v_stride, float* state, const float* decay,
+static int launch_scan_r(const float* q, const float* k, int qk_stride, const void* v, int v_stride, float* state, const float* decay,
                          float* o, const int* cu_q, const int* seq_slot, int B, int heads, int dim, int vdim, cudaStream_t st) {
     const size_t smem = (size_t)(2 * RT_TOK * dim + RT_TOK * RT_COLS) * sizeof(float);
     dim3 grid(B, heads, (vdim + RT_COLS - 1) / RT_COLS);
-    rf_launch(retention_scan_kernel<T, R>, grid, dim3(RT_COLS * 32), smem, st, q, k, reinterpret_cast<const T*>(v), v_stride, state,
+    rf_launch(retention_scan_kernel<T, R>, grid, dim3(RT_COLS * 32), smem, st, q, k, qk_stride, reinterpret_cast<const T*>(v), v_stride, state,
               decay, o, cu_q, seq_slot, heads, dim, vdim);
     RF_LAUNCH_CHECK();
     return 0;
 }
 
 template <typename T>
-static int launch_scan(const float* q, const float* k, const void* v, int v_stride, float* state, const float* decay,
+static int launch_scan(const float* q, const float* k, int qk_stride, const void* v, int v_stride, float* state, const float* decay,
                        float* o, const int* cu_q, const int* seq_slot, int B, int heads, int dim, int vdim, cudaStream_t st) {
     if (B <= 0) return 0;
     if (dim <= 0 || dim > 256 || vdim <= 0 || heads <= 0 || heads > 65535 || (vdim + RT_COLS - 1) / RT_COLS > 65535)
         return RF_ERR_UNSUPPORTED;
     switch ((dim + 31) / 32) {
-        case 1: return launch_scan_r<T, 1>(q, k, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
-        case 2: return launch_scan_r<T, 2>(q, k, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
-        case 3: return launch_scan_r<T, 3>(q, k, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
-        case 4: return launch_scan_r<T, 4>(q, k, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
-        case 5: case 6: return launch_scan_r<T, 6>(q, k, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
-        default: return launch_scan_r<T, 8>(q, k, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
+        case 1: return launch_scan_r<T, 1>(q, k, qk_stride, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
+        case 2: return launch_scan_r<T, 2>(q, k, qk_stride, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
+        case 3: return launch_scan_r<T, 3>(q, k, qk_stride, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
+        case 4: return launch_scan_r<T, 4>(q, k, qk_stride, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
+        case 5: case 6: return launch_scan_r<T, 6>(q, k, qk_stride, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
+        default: return launch_scan_r<T, 8>(q, k, qk_stride, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
     }
 }
 
@@ -444,6 +509,35 @@ static int launch_gate(const float* o, const void* gate, int gate_stride, void* 
     return 0;
 }
 
+template <typename T>
+static int launch_silu_columns(const void* src, int n_partials, long long part_stride, int row_stride, float* out, int W, int T_,
+                               cudaStream_t st) {
+    if (T_ <= 0) return 0;
+    if (W <= 0 || n_partials < 0) return RF_ERR_BAD_ARG;
+    const bool vec = W % 4 == 0 && row_stride % 4 == 0 && part_stride % 4 == 0 && !(reinterpret_cast<uintptr_t>(src) & 15) &&
+                     !(reinterpret_cast<uintptr_t>(out) & 15);
+    const size_t n = (size_t)T_ * (vec ? W / 4 : W), blocks = (n + 255) / 256;
+    const dim3 grid((unsigned)(blocks > 148 * 16 ? 148 * 16 : blocks));
+    if (vec) rf_launch(silu_columns_kernel<T, 4>, grid, dim3(256), 0, st, src, n_partials, part_stride, row_stride, out, W, n);
+    else rf_launch(silu_columns_kernel<T, 1>, grid, dim3(256), 0, st, src, n_partials, part_stride, row_stride, out, W, n);
+    RF_LAUNCH_CHECK();
+    return 0;
+}
+
+template <typename T>
+static int launch_row_norm_gate(const float* o, const void* gate, int n_partials, long long part_stride, int gate_stride, void* out,
+                                int W, float eps, const void* w, int w_is_f32, int sigmoid, int T_, cudaStream_t st) {
+    if (T_ <= 0) return 0;
+    if (W <= 0 || w == nullptr || n_partials < 0) return RF_ERR_BAD_ARG;
+    int threads = (W + 31) / 32 * 32;
+    const int most = T_ <= 296 ? 1024 : 256;
+    if (threads > most) threads = most;
+    rf_launch(row_norm_gate_kernel<T>, dim3(T_), dim3(threads), 0, st, o, gate, n_partials, part_stride, gate_stride,
+              reinterpret_cast<T*>(out), W, eps, w, w_is_f32, sigmoid);
+    RF_LAUNCH_CHECK();
+    return 0;
+}
+
 // dtype: 0 = float32, 1 = bfloat16 (of the projection's output, of v, of the gate and of the gated result)
 extern "C" {
 int rf_retention_prepare(int dtype, const void* src, int row_stride, int q_col, int k_col, float* qk, int heads, int dim,
@@ -451,18 +545,19 @@ int rf_retention_prepare(int dtype, const void* src, int row_stride, int q_col, 
     return dtype == 0 ? launch_prepare<float>(src, row_stride, q_col, k_col, qk, heads, dim, rot_dim, inv_freq, tok_pos, k_scale, T_, st)
                       : launch_prepare<__nv_bfloat16>(src, row_stride, q_col, k_col, qk, heads, dim, rot_dim, inv_freq, tok_pos, k_scale, T_, st);
 }
-int rf_retention_scan(int dtype, const float* q, const float* k, const void* v, int v_stride, float* state, const float* decay,
+// q, k float: head h's elements at columns h*dim of rows qk_stride apart
+int rf_retention_scan(int dtype, const float* q, const float* k, int qk_stride, const void* v, int v_stride, float* state, const float* decay,
                       float* o, const int* cu_q, const int* seq_slot, int B, int heads, int dim, int vdim, cudaStream_t st) {
-    return dtype == 0 ? launch_scan<float>(q, k, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st)
-                      : launch_scan<__nv_bfloat16>(q, k, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
+    return dtype == 0 ? launch_scan<float>(q, k, qk_stride, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st)
+                      : launch_scan<__nv_bfloat16>(q, k, qk_stride, v, v_stride, state, decay, o, cu_q, seq_slot, B, heads, dim, vdim, st);
 }
 // The recurrence of a prompt step in chunks of 64 tokens (see above).  LS: scratch float [n_chunks, heads, dim, vdim];
 // table: first[B+1], then n_chunks pairs (sequence, first row of the chunk among the sequence's new tokens).
-int rf_retention_chunked(int dtype, const float* q, const float* k, const void* v, int v_stride, float* state, const float* decay,
+int rf_retention_chunked(int dtype, const float* q, const float* k, int qk_stride, const void* v, int v_stride, float* state, const float* decay,
                          float* o, float* LS, const int* table, int n_chunks, const int* cu_q, const int* seq_slot, int B,
                          int heads, int dim, int vdim, cudaStream_t st) {
-    return dtype == 0 ? launch_chunked<float>(q, k, v, v_stride, state, decay, o, LS, table, n_chunks, cu_q, seq_slot, B, heads, dim, vdim, st)
-                      : launch_chunked<__nv_bfloat16>(q, k, v, v_stride, state, decay, o, LS, table, n_chunks, cu_q, seq_slot, B, heads, dim, vdim, st);
+    return dtype == 0 ? launch_chunked<float>(q, k, qk_stride, v, v_stride, state, decay, o, LS, table, n_chunks, cu_q, seq_slot, B, heads, dim, vdim, st)
+                      : launch_chunked<__nv_bfloat16>(q, k, qk_stride, v, v_stride, state, decay, o, LS, table, n_chunks, cu_q, seq_slot, B, heads, dim, vdim, st);
 }
 int rf_retention_gate(int dtype, const float* o, const void* gate, int gate_stride, void* out, int heads, int vdim, float eps,
                       int T_, cudaStream_t st) {
@@ -484,5 +579,18 @@ int rf_retention_gate_x(int dtype, const float* o, const void* gate, int gate_st
     if ((qn == nullptr) != (mt == nullptr)) return RF_ERR_BAD_ARG;
     return dtype == 0 ? launch_gate<float>(o, gate, gate_stride, out, heads, vdim, eps, T_, st, w, w_is_f32, w_per_head, sigmoid, qn, mt)
                       : launch_gate<__nv_bfloat16>(o, gate, gate_stride, out, heads, vdim, eps, T_, st, w, w_is_f32, w_per_head, sigmoid, qn, mt);
+}
+// See silu_columns_kernel: src rows of row_stride in dtype, or (n_partials > 0) float partial sums part_stride apart.
+int rf_silu_columns(int dtype, const void* src, int n_partials, long long part_stride, int row_stride, float* out, int W, int T_,
+                    cudaStream_t st) {
+    return dtype == 0 ? launch_silu_columns<float>(src, n_partials, part_stride, row_stride, out, W, T_, st)
+                      : launch_silu_columns<__nv_bfloat16>(src, n_partials, part_stride, row_stride, out, W, T_, st);
+}
+// See row_norm_gate_kernel; dtype of out, and of the gate unless it comes as partial sums.
+int rf_row_norm_gate(int dtype, const float* o, const void* gate, int n_partials, long long part_stride, int gate_stride, void* out,
+                     int W, float eps, const void* w, int w_is_f32, int sigmoid, int T_, cudaStream_t st) {
+    return dtype == 0
+        ? launch_row_norm_gate<float>(o, gate, n_partials, part_stride, gate_stride, out, W, eps, w, w_is_f32, sigmoid, T_, st)
+        : launch_row_norm_gate<__nv_bfloat16>(o, gate, n_partials, part_stride, gate_stride, out, W, eps, w, w_is_f32, sigmoid, T_, st);
 }
 }

@@ -10,7 +10,9 @@
 #define TC_THREADS 192
 #define TC_WAIT_LIMIT_NS 2000000000ULL      // 2 s
 
-enum { EPI_STORE = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_PARTIAL = 4, EPI_RESNORM = 5, EPI_CLAMPGLU = 6, EPI_REGLU = 7 };
+enum { EPI_STORE = 0, EPI_F32 = 1, EPI_RESIDUAL = 2, EPI_SWIGLU = 3, EPI_PARTIAL = 4, EPI_RESNORM = 5, EPI_CLAMPGLU = 6, EPI_REGLU = 7, EPI_GEGLU = 8 };
+// the modes whose output is half as wide as the (row-interleaved gate/up) weight
+__host__ __device__ __forceinline__ bool epi_gated(int mode) { return mode == EPI_SWIGLU || mode == EPI_CLAMPGLU || mode == EPI_REGLU || mode == EPI_GEGLU; }
 
 // What the weights-as-rows kernel needs to finish a residual update and prepare the norm that follows it
 // (mode EPI_RESNORM), and to apply a norm that was prepared that way to its own input (ss_in).
@@ -38,10 +40,13 @@ struct TcParams {
     int ldo;                // row stride of out, in elements
     int mode;
     int k_blocks_per_split; // in units of TC_BK
+    float limit;            // EPI_CLAMPGLU's constants (they fill the struct's two gaps: its size is as without them)
     long long partial_stride;   // elements between the partial sums of two splits
     int* status;            // device word: 0 = fine
     int splits;             // clustered kernel: K parts of the residual epilogue, added in order (1 = none)
+    float alpha;
 };
+static_assert(sizeof(TcParams) == 72, "a larger parameter block makes short products slower, see below");
 // (TcNorm travels as a kernel parameter of its own, and only to the kernel variant that uses it.  Inside TcParams it
 // took the kernel's parameters from 328 to 416 bytes, and every product of few tokens then needed about 4 us longer:
 // measured on the 0.5B shape, a decode step of 1.14 ms became 1.45 ms; up to 384 bytes nothing changes, from 400 on
@@ -276,27 +281,48 @@ __device__ __forceinline__ void add_bias_columns(float* v, const void* bias, int
         if (n0 + j < N) v[j] += load_vec(bias, is_f32, n0 + j);
 }
 
+// gelu by tanh: 0.5 z (1 + tanh(y)) = z / (1 + exp(-2 y)) with y = sqrt(2/pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+    return __fdividef(z, 1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float clamped_glu_fast(float g, float u, float sc, float limit, float alpha) {
+    g = fminf(g * sc, limit);
+    u = fminf(fmaxf(u * sc, -limit), limit);
+    return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);
+}
+// The gated units beside silu, from a gate and an up value in 32-bit: calls ``with`` with the unit of the mode as a function
+// (gate, up) -> value, so that the mode is settled once and not per element.
+template <typename F>
+__device__ __forceinline__ void with_gated_unit(int mode, float limit, float alpha, F&& with) {
+    if (mode == EPI_REGLU) with([](float g, float u) { return fmaxf(g, 0.f) * u; });
+    else if (mode == EPI_GEGLU) with([](float g, float u) { return gelu_tanh_fast(g) * u; });
+    else with([limit, alpha](float g, float u) { return clamped_glu_fast(g, u, 1.f, limit, alpha); });
+}
+
 template <int CH>
 __device__ __forceinline__ void epilogue_rows(const TcParams& p, const uint32_t* r, int m, int n0) {
     if (m >= p.M) return;
     const bool whole = n0 + CH <= p.N;
-    if (p.mode == EPI_REGLU) {                       // relu(gate) * up on row-interleaved gate/up columns
+    if (epi_gated(p.mode) && p.mode != EPI_SWIGLU) { // another unit on row-interleaved gate/up columns
         __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)m * p.ldo + (n0 >> 1);
-        if (whole && !(reinterpret_cast<uintptr_t>(o) & 15)) {
+        const bool vec = whole && !(reinterpret_cast<uintptr_t>(o) & 15);
+        with_gated_unit(p.mode, p.limit, p.alpha, [&](auto unit) {
+            if (vec) {
 #pragma unroll
-            for (int j = 0; j < CH; j += 16) {
-                uint32_t w[4];
+                for (int j = 0; j < CH; j += 16) {
+                    uint32_t w[4];
 #pragma unroll
-                for (int q = 0; q < 4; ++q)
-                    w[q] = pack_bf16x2(fmaxf(__uint_as_float(r[j + 4 * q]), 0.f) * __uint_as_float(r[j + 4 * q + 1]),
-                                       fmaxf(__uint_as_float(r[j + 4 * q + 2]), 0.f) * __uint_as_float(r[j + 4 * q + 3]));
-                *reinterpret_cast<uint4*>(o + (j >> 1)) = make_uint4(w[0], w[1], w[2], w[3]);
+                    for (int q = 0; q < 4; ++q)
+                        w[q] = pack_bf16x2(unit(__uint_as_float(r[j + 4 * q]), __uint_as_float(r[j + 4 * q + 1])),
+                                           unit(__uint_as_float(r[j + 4 * q + 2]), __uint_as_float(r[j + 4 * q + 3])));
+                    *reinterpret_cast<uint4*>(o + (j >> 1)) = make_uint4(w[0], w[1], w[2], w[3]);
+                }
+                return;
             }
-            return;
-        }
 #pragma unroll
-        for (int j = 0; j < CH; j += 2)
-            if (n0 + j + 1 < p.N) o[j >> 1] = __float2bfloat16_rn(fmaxf(__uint_as_float(r[j]), 0.f) * __uint_as_float(r[j + 1]));
+            for (int j = 0; j < CH; j += 2)
+                if (n0 + j + 1 < p.N) o[j >> 1] = __float2bfloat16_rn(unit(__uint_as_float(r[j]), __uint_as_float(r[j + 1])));
+        });
         return;
     }
     if (p.mode == EPI_SWIGLU) {
@@ -361,11 +387,6 @@ __device__ __forceinline__ void epilogue_rows(const TcParams& p, const uint32_t*
 
 // The gated unit with clamped halves on row-interleaved gate/up columns (EPI_CLAMPGLU): lane = row m, registers = CH
 // consecutive columns.  The row's scale is applied to the 32-bit sums before anything is clamped.
-__device__ __forceinline__ float clamped_glu_fast(float g, float u, float sc, float limit, float alpha) {
-    g = fminf(g * sc, limit);
-    u = fminf(fmaxf(u * sc, -limit), limit);
-    return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);
-}
 template <int CH>
 __device__ __forceinline__ void epilogue_clamped_glu(const TcParams& p, const uint32_t* r, int m, int n0,
                                                      const float* row_scale, float limit, float alpha) {

@@ -156,17 +156,19 @@ class StepContext:
         stream.flush()
         kernels.gemm_simt(x, w, bias, out=stream.h, accumulate=True)
 
-    def gated_activation(self, y, gate_up, activation: str = "silu"):
-        """silu(gate) * up (or relu(gate) * up) from the fused, row-interleaved gate/up matrix."""
+    def gated_activation(self, y, gate_up, activation: str = "silu", limit: float = 0.0, alpha: float = 0.0):
+        """act(gate) * up from the fused, row-interleaved gate/up matrix (act = silu, relu or gelu_tanh), or "clamped_glu":
+        g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
         tc = kernels.tensor_core
         w = gate_up.weight
-        mode = {"silu": tc.SWIGLU, "relu": tc.REGLU}[activation]
+        mode = {"silu": tc.SWIGLU, "relu": tc.REGLU, "gelu_tanh": tc.GEGLU, "clamped_glu": tc.CLAMPGLU}[activation]
+        glu = dict(limit=limit, alpha=alpha) if mode == tc.CLAMPGLU else {}
         y, row_ss = self.unpack_rows(y, w, mode)
         if gate_up.bias is None and self.uses_tensor_cores(y, w, mode):
             if y.shape[0] <= tc.SKINNY_MAX_TOKENS:
-                return tc.gemm_tc_skinny(y, w, mode=mode, row_ss=row_ss)
-            return tc.gemm_tc(y, w, mode=mode)
+                return tc.gemm_tc_skinny(y, w, mode=mode, row_ss=row_ss, **glu)
+            return tc.gemm_tc(y, w, mode=mode, **glu)
         if row_ss is not None:
             y = ScaledRows(y, row_ss[0], row_ss[1], w.shape[1]).materialize()
         gu = self.matmul(y, w, gate_up.bias)
-        return kernels.swiglu(gu, activation=activation)
+        return kernels.clamped_glu(gu, limit, alpha) if mode == tc.CLAMPGLU else kernels.swiglu(gu, activation=activation)

@@ -57,6 +57,7 @@ class ModelSpec:
     pass_offsets_prefix: str = ""
     positions: Optional[Part] = None                 # parts.embedding.LearnedPositions: a learned vector per position, added to the embedding
     positions_prefix: str = ""
+    shared: Dict[str, Part] = field(default_factory=dict)   # {prefix: part} that several blocks read (a table of per-layer token inputs)
     streams: Optional[int] = None                    # several residual streams (parts.streams): ``stream.h`` is then [T, streams, width]
 
     def named_parts(self) -> Dict[str, Part]:
@@ -66,6 +67,7 @@ class ModelSpec:
             out[self.pass_offsets_prefix] = self.pass_offsets
         if self.positions is not None:
             out[self.positions_prefix] = self.positions
+        out.update(self.shared)
         for prefix, block in zip(self.block_prefixes, self.blocks):
             for sub, part in block.sub_parts().items():
                 out[prefix + sub] = part

@@ -11,5 +11,7 @@ from .basic import (dyt_rows, scaled_add, softcap_, gated_scan, gated_chunked, m
 from .basic import (weighted_add, stretch_norm, delta_prepare, delta_scan)
 from .latent import (streams_update, pair_embed, scale_, latent_write, latent_gather, head_product, attention_latent_prefill,
                      attention_latent_prefill_supported, attention_latent_decode, attention_latent_decode_groups)
+from .basic import (silu_columns, row_norm_gate, moe_route_grouped, moe_sort_passive)
+from .layernorm import (stream_update, side_gate, RoutedSum, GatedRows)
 from ._ffi import launch_count
 from . import tensor_core

@@ -201,15 +201,18 @@ def rope_kv_write(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: in
     return q_out
 
 
+_GATED_UNITS = {"silu": "rf_swiglu", "relu": "rf_reglu", "gelu_tanh": "rf_geglu"}
+
+
 def swiglu(gu: torch.Tensor, out: torch.Tensor | None = None, activation: str = "silu") -> torch.Tensor:
-    """a[t, j] = silu(gu[t, 2j]) * gu[t, 2j+1] (``activation`` "relu": relu instead of silu)."""
-    need(activation in ("silu", "relu"), f"swiglu: activation {activation!r} (silu, relu)")
+    """a[t, j] = silu(gu[t, 2j]) * gu[t, 2j+1] (``activation`` "relu", "gelu_tanh": that function instead of silu)."""
+    need(activation in _GATED_UNITS, f"swiglu: activation {activation!r} (known: {sorted(_GATED_UNITS)})")
     need_cuda(gu)
     need(gu.dim() == 2 and gu.is_contiguous() and gu.shape[1] % 2 == 0, "swiglu: input must be [T, 2I]")
     T, I2 = gu.shape
     if out is None:
         out = torch.empty((T, I2 // 2), dtype=gu.dtype, device=gu.device)
-    f = _f("elementwise", "rf_swiglu" if activation == "silu" else "rf_reglu", c_int, c_void_p, c_void_p, c_int, c_int, c_void_p)
+    f = _f("elementwise", _GATED_UNITS[activation], c_int, c_void_p, c_void_p, c_int, c_int, c_void_p)
     check(f(dtype_code(gu.dtype), ptr(gu), ptr(out), T, I2 // 2, stream()), "swiglu")
     return out
 
@@ -787,24 +790,33 @@ def retention_prepare(proj: torch.Tensor, q_col: int, k_col: int, heads: int, di
     return qk
 
 
-def retention_scan(qk: torch.Tensor, v: torch.Tensor, state: torch.Tensor, decay: torch.Tensor, cu_q: torch.Tensor,
+def _q_and_k(qk, heads: int, dim: int, what: str):
+    """(q, k, row stride) of the recurrence's inputs: a float32 [2, T, heads*dim] tensor, or a pair of [T, heads*dim] views
+    whose rows lie equally far apart."""
+    q, k = qk[0], qk[1]
+    need(q.dtype == torch.float32 and k.dtype == torch.float32 and q.dim() == 2 and q.shape == k.shape and q.shape[1] == heads * dim
+         and q.stride(1) == 1 and k.stride(1) == 1 and q.stride(0) == k.stride(0), f"{what}: bad q/k")
+    return q, k, q.stride(0)
+
+
+def retention_scan(qk, v: torch.Tensor, state: torch.Tensor, decay: torch.Tensor, cu_q: torch.Tensor,
                    seq_slot: torch.Tensor, heads: int, dim: int, vdim: int) -> torch.Tensor:
     """S <- decay_h S + k v^T, o = S^T q, token by token for every sequence of the step; ``state`` [slots, heads, vdim,
     dim] float32 (S transposed: a value dimension's column is contiguous) is read at the step's start and left as after
     its last token.  ``v`` is a [T, heads*vdim] view (rows
     may be strided).  Returns o float32 [T, heads*vdim]."""
-    need_cuda(qk, v, state, decay, cu_q, seq_slot)
-    T = qk.shape[1]
-    need(qk.dtype == torch.float32 and qk.is_contiguous() and qk.shape == (2, T, heads * dim), "retention_scan: bad q/k")
+    q, k, qk_stride = _q_and_k(qk, heads, dim, "retention_scan")
+    need_cuda(q, k, v, state, decay, cu_q, seq_slot)
+    T = q.shape[0]
     need(v.shape == (T, heads * vdim) and v.stride(1) == 1, "retention_scan: v must be [T, heads*vdim]")
     need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, vdim, dim),
          "retention_scan: state must be float32 [slots, heads, vdim, dim]")
     need(decay.dtype == torch.float32 and decay.shape == (heads,), "retention_scan: decay must be float32 [heads]")
     B = seq_slot.shape[0]
-    o = torch.empty((T, heads * vdim), dtype=torch.float32, device=qk.device)
-    f = _f("retention", "rf_retention_scan", c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+    o = torch.empty((T, heads * vdim), dtype=torch.float32, device=q.device)
+    f = _f("retention", "rf_retention_scan", c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
            c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p)
-    check(f(dtype_code(v.dtype), ptr(qk[0]), ptr(qk[1]), ptr(v), v.stride(0), ptr(state), ptr(decay), ptr(o), ptr(cu_q),
+    check(f(dtype_code(v.dtype), ptr(q), ptr(k), qk_stride, ptr(v), v.stride(0), ptr(state), ptr(decay), ptr(o), ptr(cu_q),
             ptr(seq_slot), B, heads, dim, vdim, stream()), f"retention_scan (heads={heads}, dim={dim}, vdim={vdim})")
     return o
 
@@ -812,16 +824,16 @@ def retention_scan(qk: torch.Tensor, v: torch.Tensor, state: torch.Tensor, decay
 RETENTION_CHUNK = 64
 
 
-def retention_chunked(qk: torch.Tensor, v: torch.Tensor, state: torch.Tensor, decay: torch.Tensor, table: torch.Tensor,
+def retention_chunked(qk, v: torch.Tensor, state: torch.Tensor, decay: torch.Tensor, table: torch.Tensor,
                       cu_q: torch.Tensor, seq_slot: torch.Tensor, heads: int, dim: int, vdim: int) -> torch.Tensor:
     """What ``retention_scan`` computes, for prompts: the recurrence in chunks of 64 tokens that run side by side (per-chunk
     sums, then the states between the chunks one after the other, then every chunk's outputs from its start state), all
     in 32-bit.  ``table``: int32, first[B+1] (index of each sequence's first chunk) followed by (sequence, first row among
     the sequence's new tokens) of every chunk, in the order of the sequences.  Differs from the scan by rounding only."""
-    need_cuda(qk, v, state, decay, table, cu_q, seq_slot)
-    T = qk.shape[1]
+    q, k, qk_stride = _q_and_k(qk, heads, dim, "retention_chunked")
+    need_cuda(q, k, v, state, decay, table, cu_q, seq_slot)
+    T = q.shape[0]
     B = seq_slot.shape[0]
-    need(qk.dtype == torch.float32 and qk.is_contiguous() and qk.shape == (2, T, heads * dim), "retention_chunked: bad q/k")
     need(v.shape == (T, heads * vdim) and v.stride(1) == 1, "retention_chunked: v must be [T, heads*vdim]")
     need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, vdim, dim),
          "retention_chunked: state must be float32 [slots, heads, vdim, dim]")
@@ -829,11 +841,11 @@ def retention_chunked(qk: torch.Tensor, v: torch.Tensor, state: torch.Tensor, de
     need(table.dtype == torch.int32 and (table.numel() - (B + 1)) % 2 == 0 and table.numel() > B + 1,
          "retention_chunked: the chunk table must hold first[B+1] and a pair per chunk")
     n_chunks = (table.numel() - (B + 1)) // 2
-    o = torch.empty((T, heads * vdim), dtype=torch.float32, device=qk.device)
-    scratch = torch.empty((n_chunks, heads, dim, vdim), dtype=torch.float32, device=qk.device)
-    f = _f("retention", "rf_retention_chunked", c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+    o = torch.empty((T, heads * vdim), dtype=torch.float32, device=q.device)
+    scratch = torch.empty((n_chunks, heads, dim, vdim), dtype=torch.float32, device=q.device)
+    f = _f("retention", "rf_retention_chunked", c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
            c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p)
-    check(f(dtype_code(v.dtype), ptr(qk[0]), ptr(qk[1]), ptr(v), v.stride(0), ptr(state), ptr(decay), ptr(o), ptr(scratch),
+    check(f(dtype_code(v.dtype), ptr(q), ptr(k), qk_stride, ptr(v), v.stride(0), ptr(state), ptr(decay), ptr(o), ptr(scratch),
             ptr(table), n_chunks, ptr(cu_q), ptr(seq_slot), B, heads, dim, vdim, stream()),
           f"retention_chunked (heads={heads}, dim={dim}, vdim={vdim})")
     return o
@@ -863,6 +875,46 @@ def retention_gate(o: torch.Tensor, gate: torch.Tensor, heads: int, vdim: int, e
     check(f(dtype_code(gate.dtype), ptr(o), ptr(gate), gate.stride(0), ptr(out), heads, vdim, float(eps), T, ptr(weight),
             int(weight is not None and weight.dtype == torch.float32), int(per_head), int(gate_fn == "sigmoid"), ptr(qn),
             ptr(mt), stream()), "retention_gate")
+    return out
+
+
+def _rows_or_parts(x: torch.Tensor, what: str):
+    """(T, width, n_partials, part_stride, row_stride) of a product's matrix [T, W] (rows may be strided) or of its float32
+    partial sums [S, T, W] (a view of some columns of a contiguous stack is fine)."""
+    if x.dim() == 3:
+        need(x.dtype == torch.float32 and x.stride(2) == 1, f"{what}: partial sums must be float32 [S, T, W]")
+        return x.shape[1], x.shape[2], x.shape[0], x.stride(0), x.stride(1)
+    need(x.dim() == 2 and x.stride(1) == 1, f"{what}: expected [T, W] rows or [S, T, W] partial sums")
+    return x.shape[0], x.shape[1], 0, 0, x.stride(0)
+
+
+def silu_columns(x: torch.Tensor) -> torch.Tensor:
+    """silu(x) as float32 [T, W], of a product's columns (``x`` [T, W]) or of its partial sums ([S, T, W], float32)."""
+    need_cuda(x)
+    T, W, S, ps, rs = _rows_or_parts(x, "silu_columns")
+    out = torch.empty((T, W), dtype=torch.float32, device=x.device)
+    f = _f("retention", "rf_silu_columns", c_int, c_void_p, c_int, c_ll, c_int, c_void_p, c_int, c_int, c_void_p)
+    check(f(dtype_code(x.dtype), ptr(x), S, ps, rs, ptr(out), W, T, stream()), "silu_columns")
+    return out
+
+
+def row_norm_gate(o: torch.Tensor, gate: torch.Tensor, eps: float, weight: torch.Tensor, compute_dtype: torch.dtype,
+                  gate_fn: str = "sigmoid") -> torch.Tensor:
+    """o / sqrt(mean(o^2) + eps) over the whole row, times ``weight`` [W], times sigmoid(gate) (``gate_fn`` "silu": silu), in
+    the compute dtype.  o float32 [T, W]; gate [T, W] in the compute dtype, or float32 partial sums [S, T, W]."""
+    need_cuda(o, gate, weight)
+    need(gate_fn in ("silu", "sigmoid"), f"row_norm_gate: gate function {gate_fn!r} (silu, sigmoid)")
+    need(o.dtype == torch.float32 and o.dim() == 2 and o.is_contiguous(), "row_norm_gate: o must be contiguous float32 [T, W]")
+    T, W = o.shape
+    Tg, Wg, S, ps, rs = _rows_or_parts(gate, "row_norm_gate")
+    need((Tg, Wg) == (T, W) and (S > 0 or gate.dtype == compute_dtype), "row_norm_gate: the gate must have o's shape")
+    need(weight.shape == (W,) and weight.is_contiguous() and weight.dtype in (torch.float32, torch.bfloat16),
+         "row_norm_gate: the norm's weight must be [W]")
+    out = torch.empty((T, W), dtype=compute_dtype, device=o.device)
+    f = _f("retention", "rf_row_norm_gate", c_int, c_void_p, c_void_p, c_int, c_ll, c_int, c_void_p, c_int, c_float, c_void_p,
+           c_int, c_int, c_int, c_void_p)
+    check(f(dtype_code(compute_dtype), ptr(o), ptr(gate), S, ps, rs, ptr(out), W, float(eps), ptr(weight),
+            int(weight.dtype == torch.float32), int(gate_fn == "sigmoid"), T, stream()), "row_norm_gate")
     return out
 
 
@@ -914,14 +966,15 @@ MOE_TILE_SMALL, MOE_TILE_LARGE = 16, 64
 MOE_TILE_TC = 128          # rows of a tile of the grouped tensor-core product
 
 
-def moe_gather(x: torch.Tensor, perm: torch.Tensor, top: int) -> torch.Tensor:
-    """out[r] = x[perm[r] // top]: the tokens' activations in the order the sort left their (token, choice) pairs in."""
-    need_cuda(x, perm)
+def moe_gather(x: torch.Tensor, perm: torch.Tensor, top: int, n_active: torch.Tensor | None = None) -> torch.Tensor:
+    """out[r] = x[perm[r] // top]: the tokens' activations in the order the sort left their (token, choice) pairs in.
+    ``n_active`` (one int32 on the device): only so many leading rows are filled."""
+    need_cuda(x, perm, n_active)
     need(x.dim() == 2 and x.stride(1) == 1 and perm.dtype == torch.int32, "moe_gather: x [T, K] and an int32 permutation")
     n, K = perm.numel(), x.shape[1]
     out = torch.empty((n, K), dtype=x.dtype, device=x.device)
-    f = _f("moe", "rf_moe_gather", c_void_p, c_ll, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p)
-    check(f(ptr(x), x.stride(0) * x.element_size(), ptr(perm), top, ptr(out), K * x.element_size(), n, stream()), "moe_gather")
+    f = _f("moe", "rf_moe_gather", c_void_p, c_ll, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p)
+    check(f(ptr(x), x.stride(0) * x.element_size(), ptr(perm), top, ptr(out), K * x.element_size(), n, ptr(n_active), stream()), "moe_gather")
     return out
 
 
@@ -942,6 +995,44 @@ def moe_route(logits: torch.Tensor, top: int, scoring: str = "softmax_of_chosen"
     f = _f("moe", "rf_moe_route_scored", c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p)
     check(f(ptr(logits), E, top, ptr(idx), ptr(w), T, MOE_SCORINGS[scoring], stream()), f"moe_route (E={E}, top={top})")
     return idx, w
+
+
+def moe_route_grouped(logits: torch.Tensor, correction: torch.Tensor, top: int, *, groups: int = 1, keep: int = 1,
+                      scale: float = 1.0):
+    """(experts int32 [T, top], weights float32 [T, top]) by s = softmax(logits) over all E columns and c = s + correction:
+    the columns form ``groups`` equal groups of neighbours, a group counts by its largest c, the ``top`` largest c inside the
+    ``keep`` best groups are chosen (of equal numbers the lower index), and weighted by s / (sum of the chosen s + 1e-20) *
+    scale.  logits float32 [T, E] (rows may be strided), correction float32 [E]."""
+    need_cuda(logits, correction)
+    need(logits.dtype == torch.float32 and logits.dim() == 2 and logits.stride(1) == 1, "moe_route_grouped: logits must be float32 [T, E]")
+    T, E = logits.shape
+    need(correction.dtype == torch.float32 and correction.shape == (E,) and correction.is_contiguous(),
+         "moe_route_grouped: the correction must be float32 [E]")
+    idx = torch.empty((T, top), dtype=torch.int32, device=logits.device)
+    w = torch.empty((T, top), dtype=torch.float32, device=logits.device)
+    f = _f("moe", "rf_moe_route_grouped", c_void_p, c_ll, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int,
+           c_void_p)
+    check(f(ptr(logits), logits.stride(0), ptr(correction), E, int(groups), int(keep), top, float(scale), ptr(idx), ptr(w), T,
+            stream()), f"moe_route_grouped (E={E}, groups={groups}, keep={keep}, top={top})")
+    return idx, w
+
+
+def moe_sort_passive(idx: torch.Tensor, n_experts: int, passive: int, tile_rows: int):
+    """As ``moe_sort`` for ``n_experts`` experts followed by ``passive`` ones that have nothing to multiply: their pairs come
+    last and get no tiles.  Returns (perm, inv, tiles, max_tiles, n_active), the last an int32 tensor [1] on the device: how
+    many sorted rows belong to experts with tiles."""
+    need_cuda(idx)
+    n, E = idx.numel(), n_experts + passive
+    max_tiles = (n + tile_rows - 1) // tile_rows + n_experts
+    dev = idx.device
+    perm = torch.empty((n,), dtype=torch.int32, device=dev)
+    inv = torch.empty((n,), dtype=torch.int32, device=dev)
+    offsets = torch.empty((E + 1,), dtype=torch.int32, device=dev)
+    tiles = torch.empty((1 + 3 * max_tiles,), dtype=torch.int32, device=dev)
+    f = _f("moe", "rf_moe_sort_passive", c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p)
+    check(f(ptr(idx), n, E, n_experts, tile_rows, ptr(perm), ptr(inv), ptr(offsets), ptr(tiles), max_tiles, stream()),
+          f"moe_sort (E={n_experts} + {passive})")
+    return perm, inv, tiles, max_tiles, offsets[n_experts:n_experts + 1]
 
 
 def moe_sort(idx: torch.Tensor, n_experts: int, tile_rows: int, weights: torch.Tensor | None = None):
@@ -970,9 +1061,10 @@ def moe_sort(idx: torch.Tensor, n_experts: int, tile_rows: int, weights: torch.T
     return perm, inv, tiles, max_tiles
 
 
-def moe_combine(y: torch.Tensor, inv: torch.Tensor, w: torch.Tensor | None, top: int | None = None) -> torch.Tensor:
+def moe_combine(y: torch.Tensor, inv: torch.Tensor, w: torch.Tensor | None, top: int | None = None, identity=None) -> torch.Tensor:
     """out[t] = sum_k w[t, k] * y[inv[t*top + k]] in the order of k; y float32 [T*top, H] in sorted order.  Without ``w``
-    (``top`` must then be given) the plain sum."""
+    (``top`` must then be given) the plain sum.  ``identity`` = (idx int32 [T, top], experts, x [T, H]): a choice whose idx is
+    not below ``experts`` contributes x[t]."""
     need_cuda(y, inv, w)
     if w is None:
         need(top is not None and top >= 1 and inv.numel() % top == 0, "moe_combine: without weights, top must be given")
@@ -982,6 +1074,16 @@ def moe_combine(y: torch.Tensor, inv: torch.Tensor, w: torch.Tensor | None, top:
     need(y.dtype == torch.float32 and y.is_contiguous() and y.shape[0] == T * top, "moe_combine: y must be float32 [T*top, H]")
     H = y.shape[1]
     out = torch.empty((T, H), dtype=torch.float32, device=y.device)
+    if identity is not None:
+        idx, experts, x = identity
+        need_cuda(idx, x)
+        need(idx.dtype == torch.int32 and idx.shape == (T, top) and idx.is_contiguous() and x.shape == (T, H) and x.stride(1) == 1,
+             "moe_combine: identity experts need idx int32 [T, top] and x [T, H]")
+        f = _f("moe", "rf_moe_combine_identity", c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int,
+               c_void_p, c_ll, c_int, c_void_p)
+        check(f(dtype_code(x.dtype), ptr(y), ptr(inv), ptr(w), ptr(out), top, H, ptr(idx), int(experts), ptr(x), x.stride(0), T,
+                stream()), "moe_combine")
+        return out
     f = _f("moe", "rf_moe_combine", c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p)
     check(f(ptr(y), ptr(inv), ptr(w), ptr(out), top, H, T, stream()), "moe_combine")
     return out
@@ -1283,15 +1385,18 @@ def delta_prepare(qkv: torch.Tensor, a: torch.Tensor, dt_bias: torch.Tensor, a_l
     ``qkv`` float32 [T, >= 2 qk_heads dim]: q heads, then k heads (the values that follow are left alone); qn = q / sqrt(sum
     q^2 + unit_eps) * q_scale and kn likewise without the scale, per head, [T, qk_heads*dim]; kq [T, qk_heads] = kn . qn;
     decay [T, heads*dim] = exp(-exp(a_log[head]) softplus(a + dt_bias)) with ``a`` float32 [T, heads*dim]; beta [T, heads] =
-    sigmoid(beta_src), ``beta_src`` a [T, heads] view of the projection's output."""
+    sigmoid(beta_src), ``beta_src`` a [T, heads] view of the projection's output.  With ``dt_bias`` [heads] the decay is one
+    number per head: ``a`` (rows may be strided) and decay are then [T, heads]."""
     need_cuda(qkv, a, dt_bias, a_log, beta_src)
     T = qkv.shape[0]
     need(qkv.dtype == torch.float32 and qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] >= 2 * qk_heads * dim,
          "delta_prepare: qkv must be float32 [T, >= 2 qk_heads dim]")
-    need(a.dtype == torch.float32 and a.shape == (T, heads * dim) and a.is_contiguous(), "delta_prepare: a must be float32 [T, heads*dim]")
-    need(dt_bias.shape == (heads * dim,) and a_log.shape == (heads,) and dt_bias.dtype == a_log.dtype and dt_bias.is_contiguous()
+    per_head = dt_bias.shape == (heads,) and dim != 1
+    nd = heads if per_head else heads * dim
+    need(a.dtype == torch.float32 and a.shape == (T, nd) and a.stride(1) == 1, "delta_prepare: a must be float32 [T, heads*dim] or [T, heads]")
+    need(dt_bias.shape == (nd,) and a_log.shape == (heads,) and dt_bias.dtype == a_log.dtype and dt_bias.is_contiguous()
          and a_log.is_contiguous() and a_log.dtype in (torch.float32, torch.bfloat16),
-         "delta_prepare: dt_bias [heads*dim] and a_log [heads] of one dtype")
+         "delta_prepare: dt_bias [heads*dim] (or [heads]) and a_log [heads] of one dtype")
     need(beta_src.shape == (T, heads) and beta_src.stride(1) == 1 and beta_src.dtype in (torch.float32, torch.bfloat16),
          "delta_prepare: beta_src must be a [T, heads] view")
     need(heads % qk_heads == 0, "delta_prepare: the q/k heads must divide the heads")
@@ -1299,13 +1404,13 @@ def delta_prepare(qkv: torch.Tensor, a: torch.Tensor, dt_bias: torch.Tensor, a_l
     qn = torch.empty((T, qk_heads * dim), dtype=torch.float32, device=dev)
     kn = torch.empty_like(qn)
     kq = torch.empty((T, qk_heads), dtype=torch.float32, device=dev)
-    decay = torch.empty((T, heads * dim), dtype=torch.float32, device=dev)
+    decay = torch.empty((T, nd), dtype=torch.float32, device=dev)
     beta = torch.empty((T, heads), dtype=torch.float32, device=dev)
-    f = _f("delta", "rf_delta_prepare", c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p,
-           c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p)
-    check(f(dtype_code(beta_src.dtype), ptr(qkv), qkv.stride(0), ptr(a), ptr(dt_bias), ptr(a_log), int(a_log.dtype == torch.float32),
+    f = _f("delta", "rf_delta_prepare", c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p,
+           c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p)
+    check(f(dtype_code(beta_src.dtype), ptr(qkv), qkv.stride(0), ptr(a), a.stride(0), ptr(dt_bias), ptr(a_log), int(a_log.dtype == torch.float32),
             ptr(beta_src), beta_src.stride(0), ptr(qn), ptr(kn), ptr(kq), ptr(decay), ptr(beta), heads, qk_heads, dim,
-            float(q_scale), float(unit_eps), T, stream()), "delta_prepare")
+            int(per_head), float(q_scale), float(unit_eps), T, stream()), "delta_prepare")
     return qn, kn, kq, decay, beta
 
 
@@ -1313,7 +1418,7 @@ def delta_scan(qn: torch.Tensor, kn: torch.Tensor, kq: torch.Tensor, decay: torc
                state: torch.Tensor, cu_q: torch.Tensor, seq_slot: torch.Tensor, heads: int, qk_heads: int, dim: int,
                vdim: int, one_token: bool = False, lanes: int = 0) -> torch.Tensor:
     """The gated delta rule, token by token for every sequence of the step, per head (head h reads q/k head h // (heads /
-    qk_heads)):  S <- diag(decay_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t.
+    qk_heads)):  S <- diag(decay_t) S (decay [T, heads*dim], or [T, heads]: one number per head);  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t.
 
     ``state`` float32 [slots, heads, dim, vdim] is read and replaced; ``v`` float32 [T, >= heads*vdim] view; returns o float32
     [T, heads*vdim].  The sums' order depends on (dim, position) alone.  ``one_token``: every sequence of the
@@ -1323,14 +1428,14 @@ def delta_scan(qn: torch.Tensor, kn: torch.Tensor, kq: torch.Tensor, decay: torc
     T = qn.shape[0]
     B = seq_slot.shape[0]
     need(all(x.dtype == torch.float32 and x.is_contiguous() for x in (qn, kn, kq, decay, beta, state)), "delta_scan: float32 inputs")
-    need(qn.shape == (T, qk_heads * dim) and kn.shape == qn.shape and kq.shape == (T, qk_heads) and decay.shape == (T, heads * dim)
+    need(qn.shape == (T, qk_heads * dim) and kn.shape == qn.shape and kq.shape == (T, qk_heads) and decay.shape in ((T, heads * dim), (T, heads))
          and beta.shape == (T, heads), "delta_scan: shapes of qn, kn, kq, decay, beta")
     need(v.dtype == torch.float32 and v.dim() == 2 and v.stride(1) == 1 and v.shape == (T, heads * vdim), "delta_scan: v must be float32 [T, heads*vdim]")
     need(tuple(state.shape[1:]) == (heads, dim, vdim), "delta_scan: state must be [slots, heads, dim, vdim]")
     need(dim <= 256, "delta_scan: at most 256 key channels a head")
     o = torch.empty((T, heads * vdim), dtype=torch.float32, device=qn.device)
     f = _f("delta", "rf_delta_scan", c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p)
+           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p)
     check(f(ptr(qn), ptr(kn), ptr(kq), ptr(decay), ptr(beta), ptr(v), v.stride(0), ptr(state), ptr(o), ptr(cu_q), ptr(seq_slot),
-            B, heads, qk_heads, dim, vdim, int(bool(one_token)), int(lanes), stream()), f"delta_scan (heads={heads}, dim={dim}, vdim={vdim})")
+            B, heads, qk_heads, dim, vdim, int(decay.shape[1] == heads and dim != 1), int(bool(one_token)), int(lanes), stream()), f"delta_scan (heads={heads}, dim={dim}, vdim={vdim})")
     return o

@@ -8,8 +8,8 @@ import torch
 
 from ._ffi import KernelError, sm_count as device_sm_count, c_float, c_int, c_ll, c_void_p, check, fn, need, need_cuda, ptr, stream
 
-STORE, F32, RESIDUAL, SWIGLU, PARTIAL, RESNORM, CLAMPGLU, REGLU = 0, 1, 2, 3, 4, 5, 6, 7
-GATED = (SWIGLU, REGLU)      # modes whose output is half as wide as the (row-interleaved) weight
+STORE, F32, RESIDUAL, SWIGLU, PARTIAL, RESNORM, CLAMPGLU, REGLU, GEGLU = 0, 1, 2, 3, 4, 5, 6, 7, 8
+GATED = (SWIGLU, REGLU, GEGLU, CLAMPGLU)      # modes whose output is half as wide as the (row-interleaved) weight
 SKINNY_MAX_TOKENS = 128     # above it the large-M kernels stream the weights better (7B shape, decode step: 128 tokens
                             # 5.09 ms skinny / 6.38 ms clustered; 192 tokens as tiles of 64: 7.78 / 6.73)
 
@@ -130,9 +130,10 @@ def part_flags(device) -> torch.Tensor:
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, *, mode: int = STORE,
             out: Optional[torch.Tensor] = None, cluster: Optional[int] = None,
-            parts: int = 0) -> torch.Tensor:
+            parts: int = 0, limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
     """Tokens as accumulator rows (any M).  STORE -> bf16 [M,N]; F32 -> f32 [M,N]; RESIDUAL: out (f32) += x w^T;
-    SWIGLU / REGLU -> bf16 [M, N/2] = silu / relu (gate) * up from row-interleaved gate/up weights.  ``parts`` (clustered kernel, RESIDUAL only):
+    SWIGLU / REGLU / GEGLU -> bf16 [M, N/2] = silu / relu / gelu (gate) * up from row-interleaved gate/up weights; CLAMPGLU: the
+    unit with clamped halves and its ``limit`` and ``alpha`` (see ``gemm_tc_grouped``).  ``parts`` (clustered kernel, RESIDUAL only):
     K parts whose sums are added one after the other, 0 = the kernel's own choice."""
     _common(x, w, bias, out)
     M, K = x.shape
@@ -149,6 +150,18 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = Non
     if cluster and not cluster_supported(M, N, K, mode):
         cluster = 0                                   # e.g. an output row stride TMA cannot store to
     need(parts == 0 or (bool(cluster) and mode == RESIDUAL), "gemm: K parts need the clustered kernel and RESIDUAL")
+    need(mode != CLAMPGLU or (limit > 0 and bias is None), "gemm: the clamped unit needs a positive limit and takes no bias")
+    if cluster and mode == CLAMPGLU:
+        f = fn("gemm_tcgen05_cluster", "rf_gemm_tc_cluster_glu",
+               [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p])
+        check(f(ptr(x), x.stride(0), ptr(w), ptr(out), out.stride(0), M, N, K, cluster, float(limit), float(alpha),
+                ptr(status_word(x.device)), stream()), f"gemm_tc_cluster ({M}x{N}x{K}, clamped unit)")
+        return out
+    if mode == CLAMPGLU:
+        f = _f("rf_gemm_tc_glu", c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p)
+        check(f(ptr(x), x.stride(0), ptr(w), ptr(out), out.stride(0), M, N, K, float(limit), float(alpha),
+                ptr(status_word(x.device)), stream()), f"gemm_tc ({M}x{N}x{K}, clamped unit)")
+        return out
     if cluster:
         f = fn("gemm_tcgen05_cluster", "rf_gemm_tc_cluster",
                [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -239,7 +252,8 @@ def _row_ss_args(row_ss, M):
 
 
 def gemm_tc_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, *, mode: int = STORE,
-                   splits: int = 1, out: Optional[torch.Tensor] = None, row_ss=None) -> torch.Tensor:
+                   splits: int = 1, out: Optional[torch.Tensor] = None, row_ss=None, limit: float = 0.0,
+                   alpha: float = 0.0) -> torch.Tensor:
     """Weights as accumulator rows, for few tokens (up to 128 in one tile).  With ``splits`` > 1 the mode must be PARTIAL and
     the result is the float32 stack [splits, M, N] of partial sums.
 
@@ -259,6 +273,14 @@ def gemm_tc_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor
         need(mode != RESIDUAL, "gemm: RESIDUAL needs the tensor to add into")
         out = torch.empty(shape, dtype=odt, device=x.device)
     need(tuple(out.shape) == shape and out.dtype == odt and out.is_contiguous(), "gemm: output has the wrong shape or dtype")
+    if mode == CLAMPGLU:
+        need(limit > 0 and bias is None, "gemm: the clamped unit needs a positive limit and takes no bias")
+        ss_ptr, ss_tiles, ss_stride, eps = _row_ss_args(row_ss, M)
+        f = _f("rf_gemm_tc_skinny_glu", c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int,
+               c_float, c_float, c_float, c_void_p, c_void_p)
+        check(f(ptr(x), x.stride(0), ptr(w), ptr(out), cols, M, N, K, ss_ptr, ss_tiles, ss_stride, eps, float(limit), float(alpha),
+                ptr(status_word(x.device)), stream()), f"gemm_tc_skinny ({M}x{N}x{K}, clamped unit)")
+        return out
     if row_ss is None:
         f = _f("rf_gemm_tc_skinny", c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
                c_int, c_int, c_void_p, c_void_p)

@@ -26,3 +26,6 @@ from .latent import LatentAttention, LatentCacheAttention
 from .delta import GatedDeltaRule
 from .embedding import PairEmbedding
 from .streams import HyperConnectedBlock, HyperConnection, StreamsNorm
+from .norm import LayerNorm
+from .block import LayerNormedBlock
+from .side import SideTable, TokenSideInput

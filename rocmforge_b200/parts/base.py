@@ -132,6 +132,11 @@ class FeedForward(Part):
         """The result as float32 [T, H] instead of an update of the stream (see Mixer.output)."""
         raise NotImplementedError(f"{type(self).__name__} does not hand out its result (only forward)")
 
+    def addends(self, ctx, y: torch.Tensor) -> list:
+        """The result as a list of what ``kernels.stream_update`` sums on the way into the stream (tensors, stacks of partial
+        sums, at most one kernels.RoutedSum, kernels.GatedRows)."""
+        return [self.output(ctx, y)]
+
 
 class Block(Part):
     """Arrangement of norm(s), mixer and feed-forward around the residual stream."""

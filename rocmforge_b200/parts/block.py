@@ -252,3 +252,67 @@ class ScaledPreNormBlock(Block):
         self._add(ctx, stream, r, self.norm2)
         y = self.norm2.forward(ctx, stream)
         self._add(ctx, stream, self.ffn.output(ctx, y), after)
+
+
+@BLOCKS.register("layernormed")
+class LayerNormedBlock(Block):
+    """x += mixer(norm1(x)); x += ffn(norm2(x)); x += side(x, token), the norms layer norms.  ``ffn`` (with ``norm2``) and ``side``
+    (a ``parts.side.TokenSideInput``) may be None.
+
+    The sub-layers hand out what they have in 32-bit (``Mixer.output``, ``FeedForward.addends``: partial sums, experts' rows not
+    yet weighted, a shared unit not yet gated), and one kernel per sub-layer (``kernels.stream_update``) forms the sum, adds it
+    into the 32-bit stream and leaves what the next reader wants: the next layer norm's result, or the stream rounded for the
+    side input.  No layer norm launches on its own but the first layer's and the final one."""
+
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm = None, ffn: FeedForward = None, side: Part = None,
+                 names: Dict[str, str] = None):
+        if (ffn is None) != (norm2 is None):
+            raise ValueError("layernormed block: ffn and norm2 come together or not at all")
+        self.norm1, self.mixer, self.norm2, self.ffn, self.side = norm1, mixer, norm2, ffn, side
+        self.names = dict(names)
+
+    def sub_parts(self) -> Dict[str, Part]:
+        out = {self.names["norm1"]: self.norm1}
+        out.update(_leaves(self.names["mixer"], self.mixer))
+        if self.ffn is not None:
+            out[self.names["norm2"]] = self.norm2
+            out.update(_leaves(self.names["ffn"], self.ffn))
+        elif self.names.get("norm2") is not None:
+            # a layer without feed-forward: a folder that stores the second norm all the same is not at fault
+            import dataclasses
+            out[""] = UnusedTensors({self.names["norm2"] + local: dataclasses.replace(spec, optional=True)
+                                     for local, spec in self.norm1.param_specs().items()})
+        if self.side is not None:
+            out[self.names["side"]] = self.side
+        return out
+
+    def entry_norm(self):
+        return self.norm1
+
+    def _update(self, ctx, stream, addends, reader, post=None):
+        """stream += the addends; what ``reader`` (a norm, the side input, or None) reads next is left in stream.prepared."""
+        from .. import kernels
+        stream.flush()
+        stream.prepared = None
+        nxt = reader.layer_params() if hasattr(reader, "layer_params") else None
+        rounded = reader is not None and reader is self.side and ctx.compute_dtype != torch.float32
+        y = kernels.stream_update(stream.h, addends, ctx.compute_dtype, post=post, next_norm=nxt, rounded=rounded)
+        if y is not None:
+            stream.prepared = (reader, y)
+
+    def forward(self, ctx, stream, cache_view):
+        after, side = stream.after_block, self.side
+        stream.next_norm = None
+        last = after if side is None else side
+        y = self.norm1.forward(ctx, stream)
+        r = self.mixer.output(ctx, y, cache_view)
+        if self.ffn is None:
+            self._update(ctx, stream, [r], last)
+        else:
+            self._update(ctx, stream, [r], self.norm2)
+            self._update(ctx, stream, self.ffn.addends(ctx, self.norm2.forward(ctx, stream)), last)
+        if side is not None:
+            prepared, stream.prepared = stream.prepared, None
+            x = prepared[1] if prepared is not None and prepared[0] is side else stream.h     # (32-bit path: the stream itself)
+            update, post = side.addend(ctx, x)
+            self._update(ctx, stream, [update], after, post=post)

@@ -32,36 +32,44 @@ class GatedDeltaRule(Mixer):
     recurrence runs token by token in prompts too, so its sums do not depend on how a prompt is cut into portions (a token
     decoded alone takes another kernel form, whose sums differ by rounding).
     ``names``: the tensors' names below the part's prefix (keys q, k, v, q_conv, k_conv, v_conv, b, a_log, dt_bias, a1, a2,
-    g1, g2, norm, o).
+    g1, g2, norm, o; a and g in place of the low-rank pairs).
+
+    What other designs change: ``decay_rank`` None: ONE decay per head, g = exp(-exp(A_log_h) softplus(W_a x + dt_bias)) with
+    W_a [heads, H] and dt_bias [heads]; W_a and W_b are then a small product of their own whose result stays 32-bit.
+    ``gate_rank`` None: the gate is one full matrix W_g x, part of the first product.  ``gate_fn`` "silu" instead of sigmoid.
     """
 
-    def __init__(self, hidden: int, n_heads: int, qk_heads: int, dim: int, vdim: int, taps: int, decay_rank: int,
-                 gate_rank: int, eps: float, *, unit_eps: float = 1e-6, q_scale: Optional[float] = None,
-                 names: Optional[Dict[str, str]] = None):
+    def __init__(self, hidden: int, n_heads: int, qk_heads: int, dim: int, vdim: int, taps: int, decay_rank: Optional[int],
+                 gate_rank: Optional[int], eps: float, *, unit_eps: float = 1e-6, q_scale: Optional[float] = None,
+                 names: Optional[Dict[str, str]] = None, gate_fn: str = "sigmoid"):
         if n_heads % qk_heads:
             raise ValueError(f"gated_delta: {n_heads} heads cannot share {qk_heads} q/k heads")
         if dim > 256:
             raise ValueError(f"gated_delta: the recurrence kernel holds at most 256 rows of a state column, got dim {dim}")
         if not 1 <= taps <= 16:
             raise ValueError(f"gated_delta: the convolution kernel takes 1 to 16 taps, got {taps}")
-        if decay_rank < 1 or gate_rank < 1:
+        if any(r is not None and r < 1 for r in (decay_rank, gate_rank)):
             raise ValueError("gated_delta: the low-rank projections need a rank of at least 1")
+        if gate_fn not in ("silu", "sigmoid"):
+            raise ValueError(f"gated_delta: gate function {gate_fn!r} (silu, sigmoid)")
+        self.gate_fn = gate_fn
         self.hidden, self.n_heads, self.qk_heads, self.dim, self.vdim = hidden, n_heads, qk_heads, dim, vdim
-        self.taps, self.decay_rank, self.gate_rank = int(taps), int(decay_rank), int(gate_rank)
+        self.taps, self.decay_rank, self.gate_rank = int(taps), decay_rank, gate_rank
         self.eps, self.unit_eps = float(eps), float(unit_eps)
         self.q_scale = float(q_scale) if q_scale is not None else float(dim) ** -0.5
         self.names = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "q_conv": "q_conv.weight",
                       "k_conv": "k_conv.weight", "v_conv": "v_conv.weight", "b": "b_proj.weight", "a_log": "A_log",
                       "dt_bias": "dt_bias", "a1": "a_proj.0.weight", "a2": "a_proj.1.weight", "g1": "g_proj.0.weight",
-                      "g2": "g_proj.1.weight", "norm": "norm.weight", "o": "o_proj.weight"}
+                      "g2": "g_proj.1.weight", "a": "a_proj.weight", "g": "g_proj.weight", "norm": "norm.weight", "o": "o_proj.weight"}
         self.names.update(names or {})
-        self.qk_size, self.v_size, self.decay_size = qk_heads * dim, n_heads * vdim, n_heads * dim
+        self.qk_size, self.v_size = qk_heads * dim, n_heads * vdim
+        self.decay_size = n_heads if decay_rank is None else n_heads * dim
         self.channels = 2 * self.qk_size + self.v_size
         self.proj: Optional[Linear] = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         n = self.names
-        return {n["q"]: ParamSpec((self.qk_size, self.hidden)), n["k"]: ParamSpec((self.qk_size, self.hidden)),
+        s = {n["q"]: ParamSpec((self.qk_size, self.hidden)), n["k"]: ParamSpec((self.qk_size, self.hidden)),
                 n["v"]: ParamSpec((self.v_size, self.hidden)),
                 # random-weights mode: taps that let earlier tokens count, decays spread between fast and slow channels
                 n["q_conv"]: ParamSpec((self.qk_size, self.taps), kind="vector", init="normal", std=0.3),
@@ -70,12 +78,19 @@ class GatedDeltaRule(Mixer):
                 n["b"]: ParamSpec((self.n_heads, self.hidden), std=0.1),
                 n["a_log"]: ParamSpec((self.n_heads,), kind="vector", init="normal", std=0.5, mean=-1.0),
                 n["dt_bias"]: ParamSpec((self.decay_size,), kind="vector", init="normal", std=1.0),
-                n["a1"]: ParamSpec((self.decay_rank, self.hidden)),
-                n["a2"]: ParamSpec((self.decay_size, self.decay_rank), std=1.0),
-                n["g1"]: ParamSpec((self.gate_rank, self.hidden)),
-                n["g2"]: ParamSpec((self.v_size, self.gate_rank), std=1.0),
                 n["norm"]: ParamSpec((self.vdim,), kind="vector", init="ones"),
                 n["o"]: ParamSpec((self.hidden, self.v_size))}
+        if self.decay_rank is None:
+            s[n["a"]] = ParamSpec((self.n_heads, self.hidden), std=0.1)
+        else:
+            s[n["a1"]] = ParamSpec((self.decay_rank, self.hidden))
+            s[n["a2"]] = ParamSpec((self.decay_size, self.decay_rank), std=1.0)
+        if self.gate_rank is None:
+            s[n["g"]] = ParamSpec((self.v_size, self.hidden))
+        else:
+            s[n["g1"]] = ParamSpec((self.gate_rank, self.hidden))
+            s[n["g2"]] = ParamSpec((self.v_size, self.gate_rank), std=1.0)
+        return s
 
     def bind(self, params, compute_dtype):
         n = self.names
@@ -88,11 +103,24 @@ class GatedDeltaRule(Mixer):
                 first = torch.cat([first, first.new_zeros((rp - rank, first.shape[1]))], dim=0)
                 second = torch.cat([second, second.new_zeros((second.shape[0], rp - rank))], dim=1)
             return first, second.contiguous(), rp
-        a1, a2, self.a_rank = padded_rank(params[n["a1"]], params[n["a2"]], self.decay_rank)
-        g1, g2, self.g_rank = padded_rank(params[n["g1"]], params[n["g2"]], self.gate_rank)
+        named = [("qkv", torch.cat([params[n["q"]], params[n["k"]], params[n["v"]]], dim=0))]
+        self.a2 = self.g2 = self.ab = None
+        if self.decay_rank is None:                           # beta and the decay: a product of 2 x heads rows, 32-bit result
+            ab = torch.cat([params[n["b"]], params[n["a"]]], dim=0)
+            pad = (-ab.shape[0]) % 8
+            self.ab = Linear(torch.cat([ab, ab.new_zeros((pad, self.hidden))], dim=0).contiguous() if pad else ab.contiguous())
+        else:
+            a1, a2, self.a_rank = padded_rank(params[n["a1"]], params[n["a2"]], self.decay_rank)
+            self.a2 = Linear(a2)
+            named += [("b", params[n["b"]]), ("a1", a1)]
+        if self.gate_rank is None:
+            named.append(("g", params[n["g"]]))
+        else:
+            g1, g2, self.g_rank = padded_rank(params[n["g1"]], params[n["g2"]], self.gate_rank)
+            self.g2 = Linear(g2)
+            named.append(("g1", g1))
         blocks, at, cols = [], 0, {}
-        for name, b in (("qkv", torch.cat([params[n["q"]], params[n["k"]], params[n["v"]]], dim=0)), ("b", params[n["b"]]),
-                        ("a1", a1), ("g1", g1)):
+        for name, b in named:
             pad = (-at) % 8                               # every block starts on a 16-byte boundary of the output rows
             if pad:
                 blocks.append(b.new_zeros((pad, self.hidden)))
@@ -104,7 +132,6 @@ class GatedDeltaRule(Mixer):
             blocks.append(blocks[0].new_zeros(((-at) % 8, self.hidden)))
         self.cols = cols
         self.proj = Linear(torch.cat(blocks, dim=0).contiguous())
-        self.a2, self.g2 = Linear(a2), Linear(g2)
         self.conv_w = torch.cat([params[n["q_conv"]], params[n["k_conv"]].to(params[n["q_conv"]].dtype),
                                  params[n["v_conv"]].to(params[n["q_conv"]].dtype)], dim=0).contiguous()
         self.conv_b = torch.zeros((self.channels,), dtype=self.conv_w.dtype, device=self.conv_w.device)      # the design has none
@@ -128,9 +155,15 @@ class GatedDeltaRule(Mixer):
         if isinstance(y, ScaledRows):
             y = y.materialize()
         c = self.cols
-        p = self.proj(ctx, y)                                                # [T, q | k | v | b | a1 | g1]
-        a = self.a2(ctx, p[:, c["a1"]:c["a1"] + self.a_rank], out_f32=True)  # [T, heads*dim], 32-bit
-        gate = self.g2(ctx, p[:, c["g1"]:c["g1"] + self.g_rank])             # [T, heads*vdim]
+        p = self.proj(ctx, y)                                                # [T, q | k | v | b | a1 | g1], or [T, q | k | v | g]
+        if self.decay_rank is None:
+            ab = self.ab(ctx, y, out_f32=True)                               # [T, b | a], 32-bit
+            b, a = ab[:, :self.n_heads], ab[:, self.n_heads:2 * self.n_heads]
+        else:
+            b = p[:, c["b"]:c["b"] + self.n_heads]
+            a = self.a2(ctx, p[:, c["a1"]:c["a1"] + self.a_rank], out_f32=True)      # [T, heads*dim], 32-bit
+        gate = (p[:, c["g"]:c["g"] + self.v_size] if self.gate_rank is None
+                else self.g2(ctx, p[:, c["g1"]:c["g1"] + self.g_rank]))      # [T, heads*vdim]
         if self.taps > 1:
             conv_state = state_view["conv"]
         else:
@@ -139,11 +172,10 @@ class GatedDeltaRule(Mixer):
             conv_state = self._no_conv_state
         qkv = kernels.conv_silu(p, c["qkv"], self.channels, conv_state, self.conv_w, self.conv_b, ctx.tok_seq, ctx.cu_q,
                                 ctx.seq_slot)                                # float32 [T, q | k | v]
-        qn, kn, kq, decay, beta = kernels.delta_prepare(qkv, a, self.dt_bias, self.a_log, p[:, c["b"]:c["b"] + self.n_heads],
-                                                        self.n_heads, self.qk_heads, self.dim, self.q_scale, self.unit_eps)
+        qn, kn, kq, decay, beta = kernels.delta_prepare(qkv, a, self.dt_bias, self.a_log, b, self.n_heads, self.qk_heads, self.dim, self.q_scale, self.unit_eps)
         o = kernels.delta_scan(qn, kn, kq, decay, beta, qkv[:, 2 * self.qk_size:], state_view["S"], ctx.cu_q, ctx.seq_slot,
                                self.n_heads, self.qk_heads, self.dim, self.vdim, one_token=ctx.is_decode)
-        return kernels.retention_gate(o, gate, self.n_heads, self.vdim, self.eps, weight=self.norm_w, gate_fn="sigmoid")
+        return kernels.retention_gate(o, gate, self.n_heads, self.vdim, self.eps, weight=self.norm_w, gate_fn=self.gate_fn)
 
     def forward(self, ctx, y, cache_view, stream):
         self.o.add_to_stream(ctx, self.gated(ctx, y, cache_view), stream)

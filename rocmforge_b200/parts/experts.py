@@ -28,13 +28,35 @@ class RoutedExperts(FeedForward):
     input by the weight instead of its output, out = sum_e expert_e(w_e y) (an expert is not linear, so the two differ;
     the products being linear, w (W y) is formed in the first product's epilogue, in 32-bit, before the activation);
     ``activation`` "clamped_glu" is g sigmoid(glu_alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+
+    ``grouped`` = dict(groups, keep, scale): s = softmax(z) over all outputs, choice scores c = s + correction (a tensor
+    ``names["correction"]``, [outputs]); the outputs form ``groups`` equal groups of neighbours, a group counts by its largest
+    c, only the ``keep`` best groups' members can be chosen; the chosen are weighted by s / (sum of the chosen s + 1e-20) *
+    scale.  ``identity``: so many more router outputs, after the experts', that stand for experts without tensors whose output
+    is the feed-forward's input (with ``grouped`` only).  ``token_gate``: the name of a tensor [1, H] that rides along as one
+    more row of the router's product; its result, one 32-bit number per token, is ``token_gate_logits`` after ``output`` /
+    ``addends`` (for a branch beside this one that is gated per token).
     """
 
     def __init__(self, hidden: int, intermediate: int, n_experts: int, top: int, *, router_bias: bool = True,
                  names: Optional[Dict[str, str]] = None, expert_prefix: str = "e", scoring: str = "softmax_of_chosen",
-                 weight_on: str = "output", activation: str = "silu", limit: Optional[float] = None, glu_alpha: float = 1.702):
-        if not 1 <= top <= n_experts:
-            raise ValueError(f"routed experts: top {top} of {n_experts} experts")
+                 weight_on: str = "output", activation: str = "silu", limit: Optional[float] = None, glu_alpha: float = 1.702,
+                 grouped: Optional[Dict[str, float]] = None, identity: int = 0, token_gate: Optional[str] = None):
+        if not 1 <= top <= n_experts + identity:
+            raise ValueError(f"routed experts: top {top} of {n_experts + identity} experts")
+        if identity < 0 or (identity and grouped is None):
+            raise ValueError("routed experts: identity experts are a number, and go with the grouped choice")
+        if grouped is not None:
+            if router_bias or weight_on != "output":
+                raise ValueError("routed experts: the grouped choice goes without a router bias and with weights on the outputs")
+            g, k = int(grouped["groups"]), int(grouped["keep"])
+            if not (g >= 1 and 1 <= k <= g and (n_experts + identity) % g == 0 and k * ((n_experts + identity) // g) >= top):
+                raise ValueError(f"routed experts: {k} of {g} groups of {n_experts + identity} outputs do not hold {top} choices")
+            grouped = dict(groups=g, keep=k, scale=float(grouped["scale"]))
+        elif token_gate is not None:
+            raise ValueError("routed experts: a token gate rides along with the grouped choice's router product")
+        self.grouped, self.identity, self.token_gate = grouped, int(identity), token_gate
+        self.token_gate_logits = None
         if scoring not in kernels.MOE_SCORINGS:
             raise ValueError(f"routed experts: scoring {scoring!r} (known: {sorted(kernels.MOE_SCORINGS)})")
         if weight_on not in ("output", "input") or activation not in ("silu", "clamped_glu"):
@@ -47,7 +69,7 @@ class RoutedExperts(FeedForward):
         self.limit, self.glu_alpha = (float(limit) if limit is not None else None), float(glu_alpha)
         self.hidden, self.intermediate, self.n_experts, self.top = hidden, intermediate, n_experts, top
         self.router_bias = router_bias
-        self.names = {"router": "router", "router_bias": "router.b", "gate": "gate", "up": "up", "down": "down"}
+        self.names = {"router": "router", "router_bias": "router.b", "correction": "correction", "gate": "gate", "up": "up", "down": "down"}
         self.names.update(names or {})
         self.expert_prefix = expert_prefix
         self.router_w = self.router_b = self.gate_up = self.down = None
@@ -57,7 +79,11 @@ class RoutedExperts(FeedForward):
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         # random-weights mode: router logits a few units apart, so that a choice rarely hangs on the last bits
-        s = {self.names["router"]: ParamSpec((self.n_experts, self.hidden), std=0.5)}
+        s = {self.names["router"]: ParamSpec((self.n_experts + self.identity, self.hidden), std=0.5)}
+        if self.grouped is not None:
+            s[self.names["correction"]] = ParamSpec((self.n_experts + self.identity,), kind="vector", init="normal", std=0.1)
+        if self.token_gate is not None:
+            s[self.token_gate] = ParamSpec((1, self.hidden))
         if self.router_bias:
             s[self.names["router_bias"]] = ParamSpec((self.n_experts,), kind="vector", init="normal", std=0.5)
         for e in range(self.n_experts):
@@ -70,6 +96,13 @@ class RoutedExperts(FeedForward):
         self.router_w = params[self.names["router"]]
         self.router_b = params[self.names["router_bias"]].to(torch.float32) if self.router_bias else None
         E, F, H = self.n_experts, self.intermediate, self.hidden
+        if self.grouped is not None:
+            self.correction = params[self.names["correction"]].to(torch.float32).contiguous()
+            blocks = [self.router_w] + ([params[self.token_gate]] if self.token_gate is not None else [])
+            rows = sum(b.shape[0] for b in blocks)
+            if rows % 8:                              # the product's float32 rows stay 16-byte aligned
+                blocks.append(self.router_w.new_zeros(((-rows) % 8, H)))
+            self.router_w = torch.cat(blocks, dim=0).contiguous()
         gu = torch.stack([torch.stack([params[self._expert(e, "gate")], params[self._expert(e, "up")]], dim=1)
                           for e in range(E)])                                # [E, F, 2, H]: row 2j = gate_j, 2j+1 = up_j
         self.gate_up = gu.reshape(E, 2 * F, H).contiguous()
@@ -81,6 +114,9 @@ class RoutedExperts(FeedForward):
     def output(self, ctx, y):
         if isinstance(y, ScaledRows):
             y = y.materialize()
+        if self.grouped is not None:
+            r = self.routed(ctx, y)
+            return kernels.moe_combine(r.y, r.inv, r.w, identity=(r.idx, r.experts, r.x) if self.identity else None)
         T = y.shape[0]
         z = ctx.matmul(y, self.router_w, self.router_b, out_f32=True)         # 32-bit sums of exact products
         idx, w = kernels.moe_route(z, self.top, self.scoring)
@@ -103,6 +139,38 @@ class RoutedExperts(FeedForward):
         a = kernels.swiglu(gu)                                                               # [n, F], sorted rows
         d = kernels.gemm_simt_grouped(a, self.down, tiles, max_tiles, rows, n, out_f32=True)
         return kernels.moe_combine(d, inv, w)
+
+    def addends(self, ctx, y):
+        return [self.routed(ctx, y)] if self.grouped is not None else [self.output(ctx, y)]
+
+    def routed(self, ctx, y):
+        """The grouped choice's result before the weighted sum (kernels.RoutedSum): whoever adds it to the stream forms it in
+        the same pass."""
+        if isinstance(y, ScaledRows):
+            y = y.materialize()
+        tc = kernels.tensor_core
+        E = self.n_experts
+        z = ctx.matmul(y, self.router_w, out_f32=True)                       # 32-bit sums of exact products
+        outputs = E + self.identity
+        self.token_gate_logits = z[:, outputs] if self.token_gate is not None else None
+        idx, w = kernels.moe_route_grouped(z[:, :outputs], self.correction, self.top, **self.grouped)
+        n = y.shape[0] * self.top
+        mode = tc.SWIGLU if self.activation == "silu" else tc.CLAMPGLU
+        use_tc = (ctx.compute_dtype == torch.bfloat16 and ctx.options.tensor_core_gemm
+                  and tc.grouped_supported(2 * self.intermediate, self.hidden, mode)
+                  and tc.grouped_supported(self.hidden, self.intermediate, tc.F32))
+        rows = kernels.MOE_TILE_TC if use_tc else (kernels.MOE_TILE_SMALL if n <= 16 * E else kernels.MOE_TILE_LARGE)
+        perm, inv, tiles, max_tiles, n_active = kernels.moe_sort_passive(idx, E, self.identity, rows)
+        if use_tc:
+            x = kernels.moe_gather(y, perm, self.top, n_active=n_active if self.identity else None)
+            glu = dict(limit=self.limit, alpha=self.glu_alpha) if mode == tc.CLAMPGLU else {}
+            a = tc.gemm_tc_grouped(x, self.gate_up, tiles, max_tiles, mode=mode, **glu)
+            d = tc.gemm_tc_grouped(a, self.down, tiles, max_tiles, mode=tc.F32)
+        else:
+            gu = kernels.gemm_simt_grouped(y, self.gate_up, tiles, max_tiles, rows, n, row_map=perm, row_div=self.top)
+            a = (kernels.clamped_glu(gu, self.limit, self.glu_alpha) if self.activation == "clamped_glu" else kernels.swiglu(gu))
+            d = kernels.gemm_simt_grouped(a, self.down, tiles, max_tiles, rows, n, out_f32=True)
+        return kernels.RoutedSum(d, inv, idx, w, y, E)
 
     def _output_general(self, ctx, y, idx, w, n):
         """Weights on the experts' inputs and/or another activation: each sorted row of the first grouped product is

@@ -97,3 +97,40 @@ class DynamicTanh(Norm):
             return prepared[1]
         stream.flush()
         return kernels.dyt_rows(stream.h, self.alpha, self.weight, self.bias, self.compute_dtype, rows=rows)
+
+
+@NORMS.register("layernorm")
+class LayerNorm(Norm):
+    """y = (x - mean(x)) / sqrt(mean((x - mean)^2) + eps) * w + b, statistics in 32-bit.  Tensors: the weight ``param_name`` and
+    ``<param_name>.b`` beside it.  Whoever updates the stream last may run it in the same pass (``layer_params``) and leave the
+    result in ``stream.prepared``."""
+
+    def __init__(self, size: int, eps: float, param_name: str = "weight"):
+        self.size, self.eps, self.param_name = size, float(eps), param_name
+        self.weight = self.bias = None
+        self.compute_dtype = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        n = self.param_name
+        return {n: ParamSpec((self.size,), kind="vector", init="ones"),
+                n + ".b": ParamSpec((self.size,), kind="vector", init="zeros")}
+
+    def bind(self, params, compute_dtype):
+        n = self.param_name
+        w, b = params[n], params[n + ".b"]
+        dt = w.dtype if w.dtype == b.dtype else torch.float32
+        self.weight, self.bias = w.to(dt).contiguous(), b.to(dt).contiguous()
+        self.compute_dtype = compute_dtype
+
+    def cuda_modules(self, compute_dtype):
+        return ["layernorm"]
+
+    def layer_params(self):
+        return (self.weight, self.bias, self.eps)
+
+    def forward(self, ctx, stream, rows=None, deferred_ok=False):
+        prepared, stream.prepared = stream.prepared, None
+        if prepared is not None and prepared[0] is self and rows is None and stream.pending is None:
+            return prepared[1]
+        stream.flush()
+        return kernels.stream_update(stream.h, [], self.compute_dtype, next_norm=self.layer_params(), rows=rows)
