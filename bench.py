@@ -516,8 +516,30 @@ def gedilorn_shape(width, layers=4):
     return ged, lud
 
 
+def dubodra_shape(width, layers=4):
+    """A Dubodra configuration with layers of the size a real model has, all heads of 128: attention over all earlier positions
+    with capped scores (half of each head rotated, a quarter as many kv heads), linear attention with a state of 128 x 128 per
+    head and a fixed decay, the gated delta rule with a state of 128 x 128 per head and 4 taps (half as many q/k heads), and
+    attention again; a dense feed-forward of 4 x width in the first layer, then 15 experts of width and an identity expert in
+    4 groups of which 2 stay open, 2 per token, plus a gated shared one; 256 numbers of token input a layer.  And the two
+    configurations of equal width, heads and depth it is nearest to here: Rifizen (capped attention beside a matrix state
+    with a fixed decay per head, dense and routed feed-forwards) and Ludusun (attention, and the delta rule in one layer)."""
+    heads = width // 128
+    kvh = max(1, heads // 4)
+    att = dict(heads=heads, kv_heads=kvh, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, rot=dict(dims=64, base=1e6))
+    lin = dict(heads=heads, dim=128, vdim=128, decay=[1.0 - 2.0 ** -(5 + 7 * h / max(1, heads - 1)) for h in range(heads)])
+    dlt = dict(heads=heads, kv_heads=max(1, heads // 2), dim=128, vdim=128, conv=4)
+    kinds = [("attention", att), ("lightning", lin), ("delta", dlt), ("attention", att)]
+    moe = dict(kind="moe", expert=dict(ff=width, limit=7.0), shared=dict(ff=width, limit=7.0),
+               router=dict(experts=15, identity=1, top=2, scale=1.5, groups=dict(count=4, keep=2)))
+    dub = dict(architecture="Dubodra", vocab=32000, width=width, norm=dict(eps=1e-6), embedding=dict(scale=2.0), logit_softcap=30.0,
+               token_side=dict(dim=256), layers=[dict(type=kinds[i % 4][0], mixer=kinds[i % 4][1],
+                                                      mlp=dict(kind="dense", ff=4 * width) if i == 0 else moe) for i in range(layers)])
+    return dub, rifizen_shape(width, layers)[0], ludusun_shape(width, layers)[0]
+
+
 def rifizen_points(pk, seed, widths=(1024, 2048), tokens=PREFILL_TOKENS, batches=(8, 64), steps=64, warmup=8,
-                   names=("rifizen", "dense"), archs=("Rifizen", "Qwen2ForCausalLM"), shapes=None):
+                   names=("rifizen", "dense"), archs=("Rifizen", "Qwen2ForCausalLM"), shapes=None, top=20):
     """Prefill and decode of one design at layer sizes of a real model, beside another at equal size (by default Rifizen
     beside the dense decoder), with the heaviest kernels of each step."""
     import torch
@@ -542,7 +564,7 @@ def rifizen_points(pk, seed, widths=(1024, 2048), tokens=PREFILL_TOKENS, batches
                 s = cache.alloc_slot()
                 model.step(cache, [StepRequest(s, prompt, [tokens - 1])])
                 cache.free_slot(s)
-            r["prefill_kernels"] = kernel_table(one_prompt)
+            r["prefill_kernels"] = kernel_table(one_prompt, top)
             del cache
             for b in batches:
                 d = decode_rate(model, random_prompts(b, PROMPT_LEN, V, seed + b), steps, warmup, check=4)
@@ -554,7 +576,7 @@ def rifizen_points(pk, seed, widths=(1024, 2048), tokens=PREFILL_TOKENS, batches
 
             def one_decode():
                 model.step(cache, [StepRequest(s, [1], [0]) for s in slots])
-            r[f"decode_b{batches[0]}_kernels"] = kernel_table(one_decode)
+            r[f"decode_b{batches[0]}_kernels"] = kernel_table(one_decode, top)
             del cache, model
             torch.cuda.empty_cache()
             point[name] = r
@@ -629,7 +651,7 @@ def main():
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the configuration (named in config)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch (quick check)")
-    ap.add_argument("--only", choices=["decode", "prefill", "ablate", "0.5b", "14b", "rifizen", "vilulorn", "figalix", "ludusun", "gedilorn"], default=None,
+    ap.add_argument("--only", choices=["decode", "prefill", "ablate", "0.5b", "14b", "rifizen", "vilulorn", "figalix", "ludusun", "gedilorn", "dubodra"], default=None,
                     help="run one phase only and print a short line (small cases for profilers)")
     ap.add_argument("--shape", choices=["7b", "0.5b", "14b"], default="7b",
                     help="layer sizes for --only decode / prefill / ablate (the full run always measures all three)")
@@ -669,6 +691,12 @@ def main():
                           "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops") if k in pk},
                           **rifizen_points(pk, args.seed, steps=min(args.steps, 64), warmup=warmup, names=("figalix", "rifizen"),
                                            archs=("Figalix", "Rifizen"), shapes=figalix_shape)}))
+        return 0
+    if args.only == "dubodra":
+        print(json.dumps({"only": "dubodra", "tokens": PREFILL_TOKENS, "prompt_len": PROMPT_LEN,
+                          "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops") if k in pk},
+                          **rifizen_points(pk, args.seed, steps=min(args.steps, 64), warmup=warmup, names=("dubodra", "rifizen", "ludusun"),
+                                           archs=("Dubodra", "Rifizen", "Ludusun"), shapes=dubodra_shape)}))
         return 0
     if args.only == "gedilorn":
         print(json.dumps({"only": "gedilorn", "tokens": PREFILL_TOKENS, "prompt_len": PROMPT_LEN,

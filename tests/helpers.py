@@ -525,3 +525,104 @@ def write_gedilorn(cfg: dict, folder: str, dtype: str = "float32") -> None:
         specs[name] = s
     dt = {"float32": torch.float32, "bfloat16": torch.bfloat16}[dtype]
     rf.write_model_folder(folder, raw, specs, cfg["seed"], dt)
+
+
+# --------------------------------------------------------------------------- Dubodra
+
+def _capped(*, heads, kv_heads, dim, vdim, scale, softcap=None, rot_dims=0, rot_base=None, mlp):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale}
+    if softcap is not None:
+        m["softcap"] = softcap
+    if rot_dims:
+        m["rot"] = {"dims": rot_dims, "base": rot_base}
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def _lightning(*, dim, vdim, decay, mlp):
+    return {"type": "lightning", "mixer": {"heads": len(decay), "dim": dim, "vdim": vdim, "decay": decay}, "mlp": mlp}
+
+
+def _delta(*, heads, kv_heads, dim, vdim, conv, mlp):
+    return {"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}, "mlp": mlp}
+
+
+def _in_groups(ff, limit, experts, top, *, scale=None, identity=None, groups=None, shared=None):
+    r = {"experts": experts, "top": top}
+    if scale is not None:
+        r["scale"] = scale
+    if identity is not None:
+        r["identity"] = identity
+    if groups is not None:
+        r["groups"] = {"count": groups[0], "keep": groups[1]}
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": r}
+    if shared is not None:
+        mlp["shared"] = {"ff": shared[0], "limit": shared[1]}
+    return mlp
+
+
+# Sizes that differ from each other in every respect: each kind of layer first in one of them, values of another size than
+# keys, one kv head for nine heads and as many as heads, delta-rule heads that share q and k and heads with their own, heads
+# rotated wholly, partly and not at all, scores and logits capped and not, decays of 0, 0.5 and 1, 1 to 7 taps, states of
+# 256 x 8 and 16 x 200, layers without feed-forward, experts with and without groups, identity experts (none, some, seven
+# beside one real expert) and a shared unit, one group kept and several, one to four choices, limits that bite and that do not,
+# token inputs of 5, 11 and 24 numbers a layer and none, embedding scales of 1 and others, a width that no tensor-core kernel takes.
+DUBODRA_A = dict(seed=61, architecture="Dubodra", vocab=96, width=64, norm={"eps": 1e-5}, embedding={"scale": 2.0}, logit_softcap=8.0,
+                 token_side={"dim": 5},
+                 layers=[_delta(heads=4, kv_heads=2, dim=24, vdim=12, conv=3,
+                                mlp=_in_groups(20, 0.7, 5, 2, scale=1.7, identity=1, groups=(3, 2), shared=(24, 1.2))),
+                         _capped(heads=4, kv_heads=2, dim=16, vdim=24, scale=0.4, softcap=5.0, rot_dims=8, rot_base=100.0, mlp=None),
+                         _lightning(dim=24, vdim=12, decay=[0.5, 1.0], mlp=_dense(40)),
+                         _capped(heads=3, kv_heads=3, dim=12, vdim=12, scale=0.3, mlp=_in_groups(16, 2.0, 7, 3))])
+DUBODRA_B = dict(seed=62, architecture="Dubodra", vocab=200, width=128, norm={"eps": 1e-6},
+                 layers=[_capped(heads=9, kv_heads=1, dim=20, vdim=12, scale=0.25, softcap=2.0, rot_dims=20, rot_base=1e4, mlp=_dense(100)),
+                         _delta(heads=3, kv_heads=3, dim=64, vdim=40, conv=1, mlp=None),
+                         _lightning(dim=100, vdim=33, decay=[0.9], mlp=_in_groups(16, 3.0, 9, 3, scale=0.5, identity=3, groups=(4, 1), shared=(8, 0.5))),
+                         _delta(heads=2, kv_heads=1, dim=16, vdim=16, conv=2, mlp=_in_groups(24, 0.4, 4, 1, identity=2, groups=(2, 1)))])
+DUBODRA_C = dict(seed=63, architecture="Dubodra", vocab=304, width=256, norm={"eps": 1e-6}, embedding={"scale": 4.0}, logit_softcap=30.0,
+                 token_side={"dim": 24},
+                 layers=[_lightning(dim=64, vdim=64, decay=[0.6, 0.95, 0.999, 0.0], mlp=_dense(320)),
+                         _capped(heads=8, kv_heads=2, dim=64, vdim=64, scale=0.2, softcap=15.0, rot_dims=32, rot_base=1e6,
+                                 mlp=_in_groups(64, 1.0, 6, 2, scale=2.5, identity=2, groups=(2, 1), shared=(96, 2.0))),
+                         _delta(heads=4, kv_heads=2, dim=32, vdim=48, conv=4, mlp=_in_groups(72, 1.5, 14, 3, scale=1.0, identity=2, groups=(4, 2))),
+                         _capped(heads=4, kv_heads=1, dim=128, vdim=128, scale=0.09, rot_dims=128, rot_base=1e4, mlp=_dense(128)),
+                         _lightning(dim=128, vdim=32, decay=[0.99, 0.8], mlp=None)])
+DUBODRA_D = dict(seed=64, architecture="Dubodra", vocab=130, width=100, norm={"eps": 1e-6}, embedding={"scale": 0.5}, token_side={"dim": 11},
+                 layers=[_delta(heads=1, kv_heads=1, dim=256, vdim=8, conv=7, mlp=_in_groups(24, 0.8, 12, 4, groups=(6, 4), shared=(16, 7.0))),
+                         _capped(heads=2, kv_heads=2, dim=64, vdim=128, scale=0.3, softcap=50.0, rot_dims=2, rot_base=10.0,
+                                 mlp=_in_groups(8, 1.0, 1, 2, identity=7, groups=(8, 2))),
+                         _lightning(dim=16, vdim=200, decay=[0.1, 0.3, 0.5, 0.7, 0.95], mlp=_dense(24))])
+DUBODRA_CONFIGS = {"DA": DUBODRA_A, "DB": DUBODRA_B, "DC": DUBODRA_C, "DD": DUBODRA_D}
+
+
+def dubodra_config(cfg: dict):
+    """(typed configuration, the dict that goes into config.json)."""
+    from rocmforge_b200.config import architecture_for
+    raw = {k: v for k, v in cfg.items() if k != "seed"}
+    return architecture_for("Dubodra").config_cls.from_dict(raw), raw
+
+
+def write_dubodra(cfg: dict, folder: str, dtype: str = "float32") -> None:
+    """Matrices with a standard deviation of 1.2 / sqrt(inputs), so that scores spread and gates are not all a half; norm weights
+    around one, not one, and biases that are not zero; corrections large beside the scores they correct, most of them negative."""
+    import dataclasses
+    import rocmforge_b200 as rf
+    from rocmforge_b200.config import architecture_for
+    c, raw = dubodra_config(cfg)
+    specs = {}
+    for name, s in architecture_for("Dubodra").build(c).param_specs().items():
+        if s.kind == "matrix":
+            std = 1.2 / s.shape[1] ** 0.5
+            if name in ("embed", "side.embed"):
+                std = 0.5
+            elif name.endswith(".router"):
+                std = 2.5 / s.shape[1] ** 0.5
+            s = dataclasses.replace(s, std=std)
+        elif name.endswith(".correction"):
+            s = dataclasses.replace(s, mean=-0.6, std=0.4)
+        elif s.init == "ones":
+            s = dataclasses.replace(s, init="normal", mean=1.0, std=0.2)
+        elif s.init == "zeros":
+            s = dataclasses.replace(s, init="normal", mean=0.05, std=0.2)
+        specs[name] = s
+    dt = {"float32": torch.float32, "bfloat16": torch.bfloat16}[dtype]
+    rf.write_model_folder(folder, raw, specs, cfg["seed"], dt)

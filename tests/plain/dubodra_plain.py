@@ -164,17 +164,33 @@ def limit_to_groups(c, count: int, keep: int):
     return g.masked_fill(~open_[:, :, None], float("-inf")).reshape(c.shape)
 
 
+def choice_margin(c, top: int, groups):
+    """[T]: how far each token's choice is from being another one: the smaller of the gaps between the last kept and the
+    first dropped group and between the last chosen and the first unchosen expert of the kept groups (infinite: no gap)."""
+    margin = torch.full((c.shape[0],), float("inf"), dtype=c.dtype)
+    if groups and groups["keep"] < groups["count"]:
+        g = c.view(c.shape[0], groups["count"], -1).max(dim=-1).values.sort(dim=-1, descending=True).values
+        margin = torch.minimum(margin, g[:, groups["keep"] - 1] - g[:, groups["keep"]])
+        c = limit_to_groups(c, groups["count"], groups["keep"])
+    if top < c.shape[1]:
+        e = c.sort(dim=-1, descending=True).values
+        margin = torch.minimum(margin, e[:, top - 1] - e[:, top])
+    return margin
+
+
 def mixture(h, W, pre, mlp, forced=None, seen=None):
     """``forced`` [T, top]: the experts to use instead of the chosen ones; ``seen`` (a list) receives the chosen ones with
-    the choice scores."""
+    their ``choice_margin``."""
     r = mlp["router"]
     s, c = scores(h, W, pre)
     groups = r.get("groups")
+    if seen is not None:
+        margin = choice_margin(c, r["top"], groups)
     if groups:
         c = limit_to_groups(c, groups["count"], groups["keep"])
     chosen = c.topk(r["top"], dim=-1).indices
     if seen is not None:
-        seen.append((chosen, c))
+        seen.append((chosen, margin))
     if forced is not None:
         chosen = forced
     w = s.gather(1, chosen)
