@@ -38,7 +38,7 @@ MODULES: Dict[str, List[str]] = {
     "mamba2": ["mamba2.cu", "common.cuh"],
     "mlstm": ["mlstm.cu", "common.cuh"],
     "layernorm": ["layernorm.cu", "common.cuh"],
-    "delta": ["delta.cu", "common.cuh"],
+    "delta": ["delta.cu", "tcgen05_common.cuh", "common.cuh"],
     "streams": ["streams.cu", "common.cuh"],
     "latent": ["latent.cu", "common.cuh"],
     "random_fill": ["random_fill.cu", "common.cuh"],

@@ -1439,3 +1439,33 @@ def delta_scan(qn: torch.Tensor, kn: torch.Tensor, kq: torch.Tensor, decay: torc
     check(f(ptr(qn), ptr(kn), ptr(kq), ptr(decay), ptr(beta), ptr(v), v.stride(0), ptr(state), ptr(o), ptr(cu_q), ptr(seq_slot),
             B, heads, qk_heads, dim, vdim, int(decay.shape[1] == heads and dim != 1), int(bool(one_token)), int(lanes), stream()), f"delta_scan (heads={heads}, dim={dim}, vdim={vdim})")
     return o
+
+
+def delta_chunked(qn: torch.Tensor, kn: torch.Tensor, decay: torch.Tensor, beta: torch.Tensor, v: torch.Tensor, state: torch.Tensor,
+                  table: torch.Tensor, cu_q: torch.Tensor, seq_slot: torch.Tensor, heads: int, qk_heads: int, dim: int,
+                  vdim: int) -> torch.Tensor:
+    """What ``delta_scan`` computes with one decay per head (decay [T, heads]), for prompts: chunks of 64 tokens whose corrected
+    values come from one triangular system each, side by side; then the states between the chunks one after the other; then
+    every chunk's outputs.  All in 32-bit.  ``table``: the chunk table of ``retention_chunked``.  Differs from the scan by
+    rounding only."""
+    need_cuda(qn, kn, decay, beta, v, state, table, cu_q, seq_slot)
+    T, B = qn.shape[0], seq_slot.shape[0]
+    need(all(x.dtype == torch.float32 and x.is_contiguous() for x in (qn, kn, decay, beta, state)), "delta_chunked: float32 inputs")
+    need(qn.shape == (T, qk_heads * dim) and kn.shape == qn.shape and decay.shape == (T, heads) and beta.shape == (T, heads),
+         "delta_chunked: shapes of qn, kn, decay [T, heads], beta [T, heads]")
+    need(v.dtype == torch.float32 and v.dim() == 2 and v.stride(1) == 1 and v.shape == (T, heads * vdim), "delta_chunked: v must be float32 [T, heads*vdim]")
+    need(tuple(state.shape[1:]) == (heads, dim, vdim) and heads % qk_heads == 0 and dim <= 256,
+         "delta_chunked: state must be [slots, heads, dim, vdim] with at most 256 key channels a head")
+    need(table.dtype == torch.int32 and (table.numel() - (B + 1)) % 2 == 0 and table.numel() > B + 1,
+         "delta_chunked: the chunk table must hold first[B+1] and a pair per chunk")
+    n_chunks = (table.numel() - (B + 1)) // 2
+    size = fn("delta", "rf_delta_chunked_scratch", [c_int] * 6)
+    size.restype = c_ll
+    scratch = torch.empty((size(n_chunks, heads, qk_heads, dim, vdim, T),), dtype=torch.float32, device=qn.device)
+    o = torch.empty((T, heads * vdim), dtype=torch.float32, device=qn.device)
+    f = _f("delta", "rf_delta_chunked", c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+           c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p)
+    from .tensor_core import status_word
+    check(f(ptr(qn), ptr(kn), ptr(decay), ptr(beta), ptr(v), v.stride(0), ptr(state), ptr(o), ptr(scratch), ptr(table), n_chunks,
+            ptr(cu_q), ptr(seq_slot), B, heads, qk_heads, dim, vdim, T, ptr(status_word(qn.device)), stream()), f"delta_chunked (heads={heads}, dim={dim}, vdim={vdim})")
+    return o

@@ -315,6 +315,71 @@ def test_per_head_decays(H, G, dim, vdim):
     assert rel(state[1].cpu(), ends[0]) < 2e-5 and rel(state[2].cpu(), ends[1]) < 2e-5 and not state[0].any()
 
 
+@pytest.mark.parametrize("H,G,dim,vdim", [(4, 2, 24, 12), (3, 3, 64, 40), (1, 1, 256, 8), (2, 1, 128, 128), (2, 2, 1, 5), (1, 1, 130, 70), (2, 1, 30, 33), (1, 1, 200, 20),
+                                          (2, 2, 128, 36)])
+def test_the_delta_rule_in_chunks(H, G, dim, vdim):
+    """Prompts in chunks of 64 against the recurrence in float64: sequences of a whole number of chunks, of one token more, of a
+    few tokens, side by side; a continued state; decays of exactly 0 and 1 and tiny ones at chunk borders; keys that repeat (the
+    system is then far from the identity)."""
+    from rocmforge_b200 import kernels
+    torch.manual_seed(dim + H)
+    lens = [129, 64, 3, 200]
+    T = sum(lens)
+    q = torch.randn(T, G * dim, device=DEV) * dim ** -0.5
+    k = P.unit_vector(torch.randn(T, G, dim, device=DEV))
+    k[20:60] = k[20:21]
+    k[150:158] = k[150:151]
+    k = k.reshape(T, G * dim).contiguous()
+    wide = torch.randn(T, 3 + H * vdim, device=DEV)
+    v = wide[:, 3:]
+    beta = torch.rand(T, H, device=DEV)
+    decay = torch.rand(T, H, device=DEV) ** 0.2
+    for t, g in ((0, 0.0), (5, 1.0), (63, 0.0), (64, 1e-30), (65, 1e-30), (128, 1.0), (193, 0.0), (260, 1.0)):
+        decay[t] = g
+    decay[300:340] = 1.0
+    starts = [sum(lens[:i]) for i in range(4)]
+    state = torch.zeros(6, H, dim, vdim, device=DEV)
+    begin = torch.randn(H, dim, vdim, device=DEV)
+    state[4] = begin
+    slots = [1, 4, 0, 3]
+
+    def reference(i):
+        a, b = starts[i], starts[i] + lens[i]
+        outs, ends = [], []
+        for h in range(H):
+            g = h // (H // G)
+            o, S = P.corrected_recurrence(q[a:b, g * dim:(g + 1) * dim].double().cpu(), k[a:b, g * dim:(g + 1) * dim].double().cpu(),
+                                          v[a:b, h * vdim:(h + 1) * vdim].double().cpu(), beta[a:b, h].double().cpu(), decay[a:b, h].double().cpu(),
+                                          begin[h].double().cpu() if slots[i] == 4 else None)
+            outs.append(o); ends.append(S)
+        return torch.cat(outs, dim=1), torch.stack(ends)
+    refs = [reference(i) for i in range(4)]
+    scan_state = state.clone()
+
+    def run(parts, cut):
+        """The sequences' tokens cut[i] .. parts[i] as one step."""
+        rows = torch.cat([torch.arange(starts[i] + cut[i], starts[i] + parts[i]) for i in range(4) if parts[i] > cut[i]]).to(DEV)
+        live = [i for i in range(4) if parts[i] > cut[i]]
+        ns = [parts[i] - cut[i] for i in live]
+        counts = [(n + 63) // 64 for n in ns]
+        table = [sum(counts[:j]) for j in range(len(live) + 1)] + [x for j, n in enumerate(ns) for r in range(0, n, 64) for x in (j, r)]
+        cu = [sum(ns[:j]) for j in range(len(ns) + 1)]
+        o = kernels.delta_chunked(q[rows], k[rows], decay[rows], beta[rows], v[rows], state, i32(*table), i32(*cu), i32(*[slots[i] for i in live]),
+                                  H, G, dim, vdim)
+        return {i: o[cu[j]:cu[j + 1]] for j, i in enumerate(live)}
+    first = run([70, 64, 3, 100], [0, 0, 0, 0])
+    second = run([129, 64, 3, 200], [70, 64, 3, 100])
+    for i in range(4):
+        got = torch.cat([first[i]] + ([second[i]] if i in second else [])).cpu()
+        assert rel(got, refs[i][0]) < 5e-5, f"sequence {i}: {rel(got, refs[i][0]):.1e}"
+        assert rel(state[slots[i]].cpu(), refs[i][1]) < 5e-5, f"state of sequence {i}"
+    assert not state[2].any() and not state[5].any()
+    kernels.tensor_core.check_status("cuda:0")
+    kq = (q.view(T, G, dim) * k.view(T, G, dim)).sum(-1).contiguous()
+    scan = kernels.delta_scan(q, k, kq, decay, beta, v, scan_state, i32(0, 129, 193, 196, 396), i32(*slots), H, G, dim, vdim)
+    assert rel(scan.cpu(), torch.cat([r[0] for r in refs])) < 5e-5
+
+
 # --------------------------------------------------------------------------- attention with capped scores, every key visible
 
 def paged(k, v, extra=2):
