@@ -79,7 +79,8 @@ template <int V, typename T> __device__ __forceinline__ void st_any(T* p, const 
     } else *p = Cvt<T>::from_f32(r.v[0]);
 }
 
-// A block per row.  V elements a thread at a time: 4 where every row starts on a 16-byte boundary, else 1.
+// A block per row.  V elements a thread at a time: 4 where every row starts on a 16-byte boundary, else 1.  (Rows of widths that the
+// kernel below does not take; the row stays in shared memory between the passes.)
 template <typename T, int V>
 __global__ void __launch_bounds__(1024)
 stream_update_kernel(float* __restrict__ h, const int* __restrict__ rows, RoutedRows rt, DenseRows dn, UpdateNorms nm,
@@ -171,6 +172,138 @@ stream_update_kernel(float* __restrict__ h, const int* __restrict__ rows, Routed
     }
 }
 
+// The same with a row in registers: NV groups of four elements a thread, asked for all at once, and one barrier a sum (every warp
+// adds the warps' sums up for itself, always by the same tree).  Rows of H = 4 * NV * threads elements at most.
+template <typename T, int NV, int MAXT>
+__global__ void __launch_bounds__(MAXT)
+stream_update_regs_kernel(float* __restrict__ h, const int* __restrict__ rows, RoutedRows rt, DenseRows dn, UpdateNorms nm,
+                          T* __restrict__ y, int H) {
+    __shared__ float red[3][32];
+    pdl_trigger();
+    const float invH = 1.f / (float)H;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5, step = blockDim.x * 4, c0 = threadIdx.x * 4;
+    auto row_sum = [&](float v, int i) {
+        v = warp_sum(v);
+        if (lane == 0) red[i][warp] = v;
+        __syncthreads();
+        return warp_sum(lane < n_warps ? red[i][lane] : 0.f);
+    };
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const size_t src = (size_t)(rows != nullptr ? rows[t] : (int)t) * H;
+    const bool adds = rt.y != nullptr || dn.p != nullptr;
+    Pack<4> m[NV], old[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = c0 + i * step;
+        m[i].v[0] = m[i].v[1] = m[i].v[2] = m[i].v[3] = 0.f;
+        old[i] = m[i];
+        if (c < H) old[i] = ld_f32<4>(h + src + c);
+    }
+    if (dn.p != nullptr) {
+        const float* p = dn.p + t * H + c0;
+#pragma unroll 4
+        for (int s = 0; s < dn.n; ++s, p += dn.part_stride) {
+#pragma unroll
+            for (int i = 0; i < NV; ++i)
+                if (c0 + i * step < H) {
+                    const Pack<4> a = ld_f32<4>(p + i * step);
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) m[i].v[u] += a.v[u];
+                }
+        }
+        if (dn.gate != nullptr) {
+            const float gate = 1.f / (1.f + expf(-dn.gate[t * dn.gate_stride]));
+#pragma unroll
+            for (int i = 0; i < NV; ++i)
+#pragma unroll
+                for (int u = 0; u < 4; ++u) m[i].v[u] *= gate;
+        }
+    }
+    if (rt.y != nullptr) {
+        Pack<4> r[NV];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) r[i].v[0] = r[i].v[1] = r[i].v[2] = r[i].v[3] = 0.f;
+        for (int k = 0; k < rt.top; ++k) {
+            const size_t pr = t * rt.top + k;
+            const float w = rt.w[pr];
+            const bool real = rt.idx[pr] < rt.experts;
+            const float* yr = rt.y + (size_t)rt.inv[pr] * H + c0;
+            const T* xr = reinterpret_cast<const T*>(rt.x) + t * rt.x_stride + c0;
+#pragma unroll
+            for (int i = 0; i < NV; ++i)
+                if (c0 + i * step < H) {
+                    const Pack<4> a = real ? ld_f32<4>(yr + i * step) : ld_any<4>(xr + i * step);
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) r[i].v[u] = fmaf(w, a.v[u], r[i].v[u]);
+                }
+        }
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+#pragma unroll
+            for (int u = 0; u < 4; ++u) m[i].v[u] = r[i].v[u] + m[i].v[u];
+    }
+    if (nm.w_post != nullptr) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+#pragma unroll
+            for (int u = 0; u < 4; ++u) ss += m[i].v[u] * m[i].v[u];
+        const float r = rsqrtf(row_sum(ss, 0) * invH + nm.post_eps);
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if (c0 + i * step < H) {
+                const Pack<4> w = ld_vec<4>(nm.w_post, nm.post_is_f32, c0 + i * step);
+#pragma unroll
+                for (int u = 0; u < 4; ++u) m[i].v[u] = fmaf(m[i].v[u] * r, w.v[u], old[i].v[u]);
+            }
+    } else {
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+#pragma unroll
+            for (int u = 0; u < 4; ++u) m[i].v[u] += old[i].v[u];
+    }
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        if (c0 + i * step < H && adds) st_f32<4>(h + src + c0 + i * step, m[i]);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) sum += m[i].v[u];
+    }
+    if (y == nullptr) return;
+    if (nm.w == nullptr) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if (c0 + i * step < H) st_any<4>(y + t * H + c0 + i * step, m[i]);
+        return;
+    }
+    const float mean = row_sum(sum, 1) * invH;
+    float dev = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+        if (c0 + i * step < H)
+#pragma unroll
+            for (int u = 0; u < 4; ++u) { const float d = m[i].v[u] - mean; dev = fmaf(d, d, dev); }
+    const float r = rsqrtf(row_sum(dev, 2) * invH + nm.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+        if (c0 + i * step < H) {
+            const Pack<4> w = ld_vec<4>(nm.w, nm.w_is_f32, c0 + i * step), b = ld_vec<4>(nm.b, nm.w_is_f32, c0 + i * step);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) m[i].v[u] = fmaf((m[i].v[u] - mean) * r, w.v[u], b.v[u]);
+            st_any<4>(y + t * H + c0 + i * step, m[i]);
+        }
+}
+
+template <typename T, int NV, int MAXT>
+static int go_regs(float* h, const int* rows, const RoutedRows& rt, const DenseRows& dn, const UpdateNorms& nm, void* y, int R, int H,
+                   cudaStream_t st) {
+    const int threads = ((H / 4 + NV - 1) / NV + 31) / 32 * 32;
+    rf_launch(stream_update_regs_kernel<T, NV, MAXT>, dim3(R), dim3(threads), 0, st, h, rows, rt, dn, nm, reinterpret_cast<T*>(y), H);
+    RF_LAUNCH_CHECK();
+    return 0;
+}
+
 template <typename T, int V>
 static int go_update(float* h, const int* rows, const RoutedRows& rt, const DenseRows& dn, const UpdateNorms& nm, void* y, int R,
                      int H, cudaStream_t st) {
@@ -203,6 +336,15 @@ static int launch_update(float* h, const int* rows, const RoutedRows& rt, const 
     auto on16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     const bool vec = H % 4 == 0 && on16(h) && on16(rt.y) && on16(rt.x) && rt.x_stride % 4 == 0 && on16(dn.p) &&
                      dn.part_stride % 4 == 0 && on16(nm.w_post) && on16(nm.w) && on16(nm.b) && on16(y);
+    if (vec && R <= 296) {                               // few rows: a group of elements a thread (the pass is a chain of loads)
+        if (H <= 4096) return go_regs<T, 1, 1024>(h, rows, rt, dn, nm, y, R, H, st);
+        if (H <= 8192) return go_regs<T, 2, 1024>(h, rows, rt, dn, nm, y, R, H, st);
+    } else if (vec) {                                    // many: small blocks, several on a multiprocessor
+        if (H <= 1024) return go_regs<T, 1, 256>(h, rows, rt, dn, nm, y, R, H, st);
+        if (H <= 2048) return go_regs<T, 2, 256>(h, rows, rt, dn, nm, y, R, H, st);
+        if (H <= 4096) return go_regs<T, 4, 256>(h, rows, rt, dn, nm, y, R, H, st);
+        if (H <= 8192) return go_regs<T, 8, 256>(h, rows, rt, dn, nm, y, R, H, st);
+    }
     return vec ? go_update<T, 4>(h, rows, rt, dn, nm, y, R, H, st) : go_update<T, 1>(h, rows, rt, dn, nm, y, R, H, st);
 }
 

@@ -27,7 +27,7 @@ def ref_layer_norm(x, w, b, eps):
     return c / torch.sqrt((c * c).mean(dim=-1, keepdim=True) + eps) * w + b
 
 
-@pytest.mark.parametrize("T,H", [(1, 64), (5, 100), (3, 33), (300, 256), (7, 2048), (320, 1030), (2, 14000)])
+@pytest.mark.parametrize("T,H", [(1, 64), (5, 100), (3, 33), (300, 256), (7, 2048), (320, 1030), (2, 14000), (3, 5000), (310, 2100), (300, 5120), (299, 1996)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_layer_norm_of_all_and_of_listed_rows(T, H, dtype):
     """A row far from zero mean (an RMS norm, or a variance taken around zero, is far off), a nearly constant one (eps counts)."""
@@ -46,7 +46,7 @@ def test_layer_norm_of_all_and_of_listed_rows(T, H, dtype):
     assert rel(y2, want[rows.long()]) < tol
 
 
-@pytest.mark.parametrize("T,H,parts", [(1, 64, 3), (4, 99, 1), (40, 256, 11), (310, 1024, 1), (3, 2048, 15)])
+@pytest.mark.parametrize("T,H,parts", [(1, 64, 3), (4, 99, 1), (40, 256, 11), (310, 1024, 1), (3, 2048, 15), (300, 1500, 2), (305, 3000, 1), (2, 4104, 3), (300, 4200, 1)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_update_sums_gates_norms_and_hands_on(T, H, parts, dtype):
     """The routed rows with identity experts, a gated stack of partial sums, both together, an update normed before it is added,
