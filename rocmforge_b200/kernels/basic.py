@@ -1441,6 +1441,13 @@ def delta_scan(qn: torch.Tensor, kn: torch.Tensor, kq: torch.Tensor, decay: torc
     return o
 
 
+@functools.lru_cache(None)
+def _delta_scratch():
+    size = fn("delta", "rf_delta_chunked_scratch", [c_int] * 6)
+    size.restype = c_ll
+    return size
+
+
 def delta_chunked(qn: torch.Tensor, kn: torch.Tensor, decay: torch.Tensor, beta: torch.Tensor, v: torch.Tensor, state: torch.Tensor,
                   table: torch.Tensor, cu_q: torch.Tensor, seq_slot: torch.Tensor, heads: int, qk_heads: int, dim: int,
                   vdim: int) -> torch.Tensor:
@@ -1459,9 +1466,7 @@ def delta_chunked(qn: torch.Tensor, kn: torch.Tensor, decay: torch.Tensor, beta:
     need(table.dtype == torch.int32 and (table.numel() - (B + 1)) % 2 == 0 and table.numel() > B + 1,
          "delta_chunked: the chunk table must hold first[B+1] and a pair per chunk")
     n_chunks = (table.numel() - (B + 1)) // 2
-    size = fn("delta", "rf_delta_chunked_scratch", [c_int] * 6)
-    size.restype = c_ll
-    scratch = torch.empty((size(n_chunks, heads, qk_heads, dim, vdim, T),), dtype=torch.float32, device=qn.device)
+    scratch = torch.empty((_delta_scratch()(n_chunks, heads, qk_heads, dim, vdim, T),), dtype=torch.float32, device=qn.device)
     o = torch.empty((T, heads * vdim), dtype=torch.float32, device=qn.device)
     f = _f("delta", "rf_delta_chunked", c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
            c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p)

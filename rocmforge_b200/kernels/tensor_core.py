@@ -57,6 +57,11 @@ def _f(name, *argtypes):
 
 
 @functools.lru_cache(None)
+def _fc(name, *argtypes):
+    return fn("gemm_tcgen05_cluster", name, list(argtypes))
+
+
+@functools.lru_cache(None)
 def supported(M: int, N: int, K: int, mode: int = STORE) -> bool:
     f = _f("rf_gemm_tc_supported", c_int, c_int, c_int, c_int)
     return bool(f(M, N, K, mode))
@@ -152,8 +157,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = Non
     need(parts == 0 or (bool(cluster) and mode == RESIDUAL), "gemm: K parts need the clustered kernel and RESIDUAL")
     need(mode != CLAMPGLU or (limit > 0 and bias is None), "gemm: the clamped unit needs a positive limit and takes no bias")
     if cluster and mode == CLAMPGLU:
-        f = fn("gemm_tcgen05_cluster", "rf_gemm_tc_cluster_glu",
-               [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p])
+        f = _fc("rf_gemm_tc_cluster_glu", c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
+                c_void_p, c_void_p)
         check(f(ptr(x), x.stride(0), ptr(w), ptr(out), out.stride(0), M, N, K, cluster, float(limit), float(alpha),
                 ptr(status_word(x.device)), stream()), f"gemm_tc_cluster ({M}x{N}x{K}, clamped unit)")
         return out
@@ -163,9 +168,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = Non
                 ptr(status_word(x.device)), stream()), f"gemm_tc ({M}x{N}x{K}, clamped unit)")
         return out
     if cluster:
-        f = fn("gemm_tcgen05_cluster", "rf_gemm_tc_cluster",
-               [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                c_int, c_void_p, c_int, c_void_p, c_void_p])
+        f = _fc("rf_gemm_tc_cluster", c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                c_int, c_void_p, c_int, c_void_p, c_void_p)
         flags = part_flags(x.device)
         check(f(ptr(x), x.stride(0), ptr(w), ptr(bias), int(bias is not None and bias.dtype == torch.float32),
                 ptr(out), out.stride(0), M, N, K, mode, cluster, parts, ptr(flags), flags.numel(),
